@@ -287,8 +287,10 @@ int32_t vx_decoder_step(vx_decoder *d, const int32_t *tokens_in,
    unpack the codes in registers instead, once for sixteen positions (the
    kernel of the grouped experts, and its fp8 twin). */
 int32_t vx_decoder_prefill(vx_decoder *d, const int32_t *tokens, int32_t count);
-/* The logits of the last step: device memory, [batch, vocab] f32. */
+/* The logits of the last step: device memory, [batch, vocab] f32, each row
+   vx_decoder_logits_pitch() values after the one before. */
 const float *vx_decoder_logits(const vx_decoder *d);
+int32_t vx_decoder_logits_pitch(const vx_decoder *d);
 /* The K (which = 0) or V (which = 1) cache of this rank: device memory, f32
    [layer][sequence][max_seq][kv_heads][head_dim], vx_decoder_kv_cache_bytes()
    bytes each. What a prefill process hands to a decode process
@@ -315,6 +317,65 @@ int32_t vx_decoder_kernels_per_step(const vx_decoder *d);
    `capacity` of them to `out` and returns how many, 0 when there are none. No
    counterpart in the reference: a measuring aid. */
 int32_t vx_decoder_step_trace(vx_decoder *d, uint64_t *out, int32_t capacity);
+
+/* ---- decoders of parallel blocks ----------------------------------------------
+ * x += mixer(h) + ff(h), h one RMSNorm of x: causal attention over a sliding
+ * window whose keys serve as values, scored without rotation, its output
+ * gated by sigmoid(W_g h); ff = W_down relu(W_up h)^2. The residual starts as an
+ * RMSNorm of scale * embedding row + sinusoid of the position. Layers may differ in
+ * every size and may name the same matrices; each has a ring of keys of its own.
+ * No counterpart in the reference. Everything that follows (vx_decoder_step,
+ * _reset, _prefill, _logits, _kv_cache, _adopt_kv, _destroy) takes such a decoder:
+ * its V cache is NULL, its K cache holds the layers' rings one after another,
+ * [sequence][rows of the ring][kv_heads][head_dim] f32, position t in row
+ * t mod rows; vx_decoder_prefill takes any number of tokens >= 1.
+ *
+ * Device pointers; the caller owns the memory. Matrices are bf16 or f32, gains
+ * f32 (what multiplies the normalised value). head_dim is a multiple of 8 of at
+ * most 512, q_heads * head_dim + hidden a multiple of 64: fill head rows, hidden
+ * rows and the matching columns up with zeros. */
+typedef struct {
+  int32_t q_heads, kv_heads, head_dim;
+  int32_t hidden; /* what q_heads * head_dim leaves of the output matrix's columns */
+  int32_t window; /* position p sees p - window + 1 .. p */
+  float score_scale;
+  const float *norm;  /* [dim] */
+  const void *w_in;   /* rows q | k | gate | up:
+                         [(2 q_heads + kv_heads) head_dim + hidden, dim] */
+  const void *w_out;  /* columns attention | up: [dim, q_heads head_dim + hidden] */
+} vx_parallel_layer;
+
+typedef struct {
+  int32_t width;      /* values of the residual */
+  int32_t dim;        /* width filled up to a multiple of 64 with zeros */
+  int32_t n_layers, vocab;
+  int32_t vocab_rows; /* vocab filled up to a multiple of 8 with rows of zeros */
+  int32_t max_seq;    /* positions a sequence may have */
+  int32_t weights_bf16; /* 1: bf16 matrices; 0: f32 ones, every product on the
+                           FP32 pipe */
+  int32_t batch;        /* 1, 2, 4, 8 or 16 sequences */
+  /* positions of a prompt that go through the layers together at most (0: 2048);
+     a ring has min(max_seq, window - 1 + this) rows */
+  int32_t prefill_rows;
+  float eps, embed_scale;
+  const void *embed;       /* [vocab_rows, dim] */
+  const void *classifier;  /* the same matrix, or another one like it */
+  const float *embed_norm, *final_norm; /* [dim] */
+  const double *turns; /* [(width + 1) / 2]: the part of a full turn that the angle
+                          of values 2i (sine) and 2i + 1 (cosine) advances per
+                          position */
+  const vx_parallel_layer *layers; /* host memory, n_layers of them */
+} vx_parallel_config;
+
+/* NULL with vx_b200_last_error() for sizes it cannot take. */
+vx_decoder *vx_decoder_create_parallel(const vx_parallel_config *config);
+/* The next `count` tokens of a one-sequence decoder of parallel blocks, and the
+   logits after n_want of them: want[i] (host, ascending) counts from the first of
+   these tokens, and row i of logits (host, [n_want, vocab] f32) belongs to it.
+   Waits for the GPU when n_want > 0. Returns count, or -1 with
+   vx_b200_last_error(). */
+int32_t vx_decoder_prefill_logits(vx_decoder *d, const int32_t *tokens, int32_t count,
+                                  const int32_t *want, int32_t n_want, float *logits);
 
 /* A llama2.c checkpoint: the file the reference's llama programs read through
    vx_load_config and vx_load_weights (stdlib/rust_core/src/ffi/llama.rs:11-47;

@@ -24,6 +24,7 @@
  * cores (rowdot_umma.cu).  vx_decoder_prefill uses the same kernels to read a
  * one-sequence prompt sixteen positions per pass.
  */
+#include "decoder_state.h"
 #include "kernels.h"
 #include "vx_b200.h"
 #include "vx_collective.h"
@@ -44,28 +45,11 @@
 
 namespace vxb {
 cudaStream_t caller_stream();
-void set_last_error(const char *why);
 void note_kernel(const char *name);
 vx::NcclCollective *nccl_job();
 } // namespace vxb
 
 namespace {
-
-[[noreturn]] void stop(const char *fmt, ...) {
-  va_list ap;
-  va_start(ap, fmt);
-  fputs("[Vx CUDA] FATAL: ", stderr);
-  vfprintf(stderr, fmt, ap);
-  fputc('\n', stderr);
-  va_end(ap);
-  abort();
-}
-#define CUDA_OK(expr)                                                          \
-  do {                                                                         \
-    const cudaError_t e_ = (expr);                                             \
-    if (e_ != cudaSuccess)                                                     \
-      stop("%s failed: %s", #expr, cudaGetErrorString(e_));                    \
-  } while (0)
 
 __global__ void advance_by_kernel(int32_t *pos, int by) {
   if (threadIdx.x == 0)
@@ -96,13 +80,6 @@ __global__ void add_kernel(float *x, const float *t, int64_t n) {
    sums -- and waits (bounded) for rank r's record of sequence b; then the
    largest value wins, the lowest index on a tie (rank order is index order, so
    the first rank with that value). One block; slots: [2 sets][ranks][batch]. */
-struct PickSlot {
-  float value;
-  int32_t index, call, call_again;
-};
-struct PickPeers {
-  PickSlot *slots[vxb::kMaxTpRanks];
-};
 __global__ void __launch_bounds__(vxb::kMaxTpRanks * 32)
 tp_pick_kernel(int32_t *token, const int32_t *local_best, const float *logits,
                int64_t stride, int vocab_offset, PickPeers peers, int ranks,
@@ -187,72 +164,7 @@ __global__ void pick_pair_kernel(int32_t *token, const float2 *gathered,
 
 } // namespace
 
-struct vx_decoder {
-  vx_decoder_config c;
-  int ranks, q_local, kv_local, hidden_local, vocab_local, vocab_offset;
-  std::vector<const void *> attn_norm, wq, wk, wv, bqkv, wo, ffn_norm, w_gate,
-      w_up, w_down, s_qkv, s_o, s_gate_up, s_down;
-  int wfmt; /* 0, or kFmtFp8 / kFmtQ4 for the layers' projections */
-  const void *embed, *final_norm, *lm_head;
-  const float *cos_t, *sin_t;
-  /* device state */
-  float *x, *xn, *q, *att, *h, *tmp, *logits, *k_cache, *v_cache, *scratch;
-  bool fused_norm; /* the activations of all sequences fit the projections' shared memory */
-  int32_t *tokens, *positions, *counters, *local_best;
-  float2 *pair, *pairs_all;
-  /* tp_reduce == 1: partial sums exchanged through peer memory */
-  bool push;
-  vxb::TpPush tp;
-  void *recv;                       /* this rank's slots + flags (IPC-shared) */
-  void *peer_recv[vxb::kMaxTpRanks];
-  int32_t *tp_epoch, *tp_done, *pick_epoch, *pick_gave_up;
-  PickPeers pick;
-  /* 8 or 16 sequences: the projections run on the tensor cores */
-  bool mma;
-  void *mma_xs;
-  float *mma_scratch;
-  /* a one-sequence decoder reading a whole prompt at once (prefill.cu):
-     activations of rows_cap positions, their bf16 terms, the GEMMs' partial
-     sums */
-  float *rows_x, *rows_q, *rows_partials;
-  void *rows_terms;
-  /* quantised weights: the matrix in hand as two (Q4_0) or three (fp8) bf16
-     terms, and the activations' terms spread over six or seven segments */
-  void *rows_w_terms, *rows_terms6;
-  size_t rows_partial_floats;
-  int32_t *rows_tokens;
-  int rows_cap;
-  int64_t cache_layer_stride, cache_batch_stride;
-  int split;
-  int host_pos;
-  cudaStream_t stream;
-  std::map<int, cudaGraphExec_t> graphs;
-  int kernels_per_step;
-  void *owned_weights; /* a checkpoint this decoder loaded itself, or NULL */
-  /* one sequence, bf16 weights, heads of 128 values: all layers and the logits
-     of a step are one cooperative launch (step_kernel.cu) */
-  bool one_kernel;
-  vxb::StepOp *step_ops;
-  int n_step_ops;
-  float *step_scratch;
-  int32_t *arrivals;
-  unsigned long long *step_trace; /* VXB_STEP_TRACE=1: clock readings of the last step */
-};
-
 namespace {
-
-void need(const char *why, const char *what) {
-  if (why)
-    stop("vx_decoder: %s: %s", what, why);
-}
-
-template <typename T> T *dev_alloc(size_t count) {
-  void *p = nullptr;
-  if (cudaMalloc(&p, count * sizeof(T)) != cudaSuccess)
-    stop("vx_decoder: out of device memory for %zu bytes", count * sizeof(T));
-  CUDA_OK(cudaMemset(p, 0, count * sizeof(T)));
-  return (T *)p;
-}
 
 void all_reduce(vx_decoder *d, float *buf, int64_t count) {
   vx::NcclCollective *job = vxb::nccl_job();
@@ -418,14 +330,16 @@ void build_step_ops(vx_decoder *d) {
   d->one_kernel = true;
 }
 
+} // namespace
+
 /* The end of a step: the token of every sequence (agreed between the ranks of
    a vocabulary-split model), then the positions move on. */
-void record_tail(vx_decoder *d, int launches) {
+void decoder_record_tail(vx_decoder *d, int launches) {
   const vx_decoder_config &c = d->c;
   const int B = c.batch;
   cudaStream_t s = d->stream;
   if (d->ranks == 1) {
-    need(vxb::argmax(d->tokens, d->logits, d->vocab_local, B, d->vocab_local, s),
+    need(vxb::argmax(d->tokens, d->logits, d->vocab_local, B, d->logit_stride, s),
          "argmax");
     launches += 1;
   } else {
@@ -454,6 +368,12 @@ void record_tail(vx_decoder *d, int launches) {
   ++launches;
   d->kernels_per_step = launches;
 }
+void decoder_advance(vx_decoder *d, int count) {
+  advance_by_kernel<<<1, 32, 0, d->stream>>>(d->positions, count);
+  d->host_pos += count;
+}
+
+namespace {
 
 /* One sequence: embed, then every layer and the logits in one launch. */
 void record_one_kernel_step(vx_decoder *d) {
@@ -481,10 +401,14 @@ void record_one_kernel_step(vx_decoder *d) {
     a.tp = d->tp;
   a.trace = d->step_trace;
   need(vxb::decode_step(a, s), "the step kernel");
-  record_tail(d, 2);
+  decoder_record_tail(d, 2);
 }
 
 void record_step(vx_decoder *d, int max_pos) {
+  if (d->par) {
+    decoder_record_parallel_step(d);
+    return;
+  }
   if (d->one_kernel) {
     record_one_kernel_step(d);
     return;
@@ -693,7 +617,7 @@ void record_step(vx_decoder *d, int max_pos) {
   need(vxb::matvec(la, s), "the logits");
   ++launches;
   }
-  record_tail(d, launches);
+  decoder_record_tail(d, launches);
 }
 
 cudaGraphExec_t graph_for(vx_decoder *d, int bucket) {
@@ -855,6 +779,8 @@ vx_decoder *vx_decoder_create(const vx_decoder_config *config,
     d->mma_scratch = dev_alloc<float>(vxb::batched_proj_scratch_floats(rows_max, B));
     d->mma = true;
   }
+  d->logit_stride = d->vocab_local;
+  d->par = nullptr;
   d->one_kernel = false;
   d->step_ops = nullptr;
   d->n_step_ops = 0;
@@ -907,6 +833,7 @@ void vx_decoder_destroy(vx_decoder *d) {
                   (void *)d->step_scratch, (void *)d->arrivals,
                   (void *)d->step_trace})
     cudaFree(p);
+  decoder_free_parallel(d);
   cudaFree(d->owned_weights);
   cudaStreamDestroy(d->stream);
   delete d;
@@ -936,7 +863,7 @@ int32_t vx_decoder_step(vx_decoder *d, const int32_t *tokens_in,
   const int pos = d->host_pos;
   if (pos >= d->c.max_seq)
     stop("vx_decoder_step: position %d is past max_seq %d", pos, d->c.max_seq);
-  cudaGraphExec_t exec = graph_for(d, d->one_kernel ? 0 : pos / 256);
+  cudaGraphExec_t exec = graph_for(d, d->one_kernel || d->par ? 0 : pos / 256);
   if (tokens_in)
     CUDA_OK(cudaMemcpyAsync(d->tokens, tokens_in, d->c.batch * sizeof(int32_t),
                             cudaMemcpyHostToDevice, d->stream));
@@ -961,6 +888,8 @@ int32_t vx_decoder_step(vx_decoder *d, const int32_t *tokens_in,
    there are fewer than 32: single steps are as fast then), or -1 with
    vx_b200_last_error() when this decoder cannot do it. */
 int32_t vx_decoder_prefill(vx_decoder *d, const int32_t *tokens, int32_t count) {
+  if (d->par)
+    return vx_decoder_prefill_logits(d, tokens, count, nullptr, 0, nullptr);
   const vx_decoder_config &c = d->c;
   const int hd = c.head_dim;
   const int qkv_rows = (d->q_local + 2 * d->kv_local) * hd, att_cols = d->q_local * hd;
@@ -1127,8 +1056,7 @@ int32_t vx_decoder_prefill(vx_decoder *d, const int32_t *tokens, int32_t count) 
            "RMSNorm");
     }
   }
-  advance_by_kernel<<<1, 32, 0, s>>>(d->positions, T);
-  d->host_pos += T;
+  decoder_advance(d, T);
   return T;
 }
 
@@ -1350,20 +1278,37 @@ float *vx_decoder_kv_cache(vx_decoder *d, int32_t which) {
   return which == 0 ? d->k_cache : which == 1 ? d->v_cache : nullptr;
 }
 
+int32_t vx_decoder_logits_pitch(const vx_decoder *d) { return d->logit_stride; }
+
 int64_t vx_decoder_kv_cache_bytes(const vx_decoder *d) {
+  if (d->par)
+    return d->par->cache_floats * (int64_t)sizeof(float);
   return d->cache_layer_stride * d->c.n_layers * (int64_t)sizeof(float);
 }
 
 int32_t vx_decoder_adopt_kv(vx_decoder *d, const float *k, const float *v,
                             int32_t positions) {
-  if (!k || !v || positions < 0 || positions > d->c.max_seq) {
+  if (!k || (!v && !d->par) || positions < 0 || positions > d->c.max_seq) {
     vxb::set_last_error("vx_decoder_adopt_kv: needs both caches and 0 <= "
                         "positions <= max_seq");
     return -1;
   }
   /* rows 0 .. positions-1 of every layer and sequence; one copy each (the
      source may be another GPU's memory: unified addressing finds the way) */
-  const size_t run = (size_t)positions * d->kv_local * d->c.head_dim * sizeof(float);
+  if (d->par) /* a ring: as many of its rows as the positions have reached */
+    for (const ParallelLayer &layer : d->par->layers) {
+      const int rows = positions < layer.cache_rows ? positions : layer.cache_rows;
+      for (int b = 0; b < d->c.batch && rows; ++b) {
+        const int64_t at = layer.cache_at + b * layer.cache_batch_stride;
+        CUDA_OK(cudaMemcpyAsync(
+            d->k_cache + at, k + at,
+            (size_t)rows * layer.kv_heads * layer.head_dim * sizeof(float),
+            cudaMemcpyDefault, d->stream));
+      }
+    }
+  const size_t run = d->par ? 0
+                            : (size_t)positions * d->kv_local * d->c.head_dim *
+                                  sizeof(float);
   for (int l = 0; l < d->c.n_layers && run; ++l)
     for (int b = 0; b < d->c.batch; ++b) {
       const int64_t at = l * d->cache_layer_stride + b * d->cache_batch_stride;

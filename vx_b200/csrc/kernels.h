@@ -81,6 +81,7 @@ struct MatvecArgs {
   const int32_t *expert_ids;
   int expert_slot, experts;
   const float *add_scale;
+  int norm_n;          /* the RMSNorm's mean is over so many values (0: cols) */
   int mode;            /* 0 y = s, 1 y += s, 2 y = s + bias,
                           3 y += the sum of all ranks' s (see TpPush) */
   const void *bias;    /* mode 2, bf16 */
@@ -172,6 +173,40 @@ struct QkvArgs {
   int max_seq;
 };
 const char *qkv_rope_store(const QkvArgs &a, cudaStream_t stream);
+
+/* ---- parallel blocks --------------------------------------------------------
+ * x += mixer(h) + ff(h) with h one norm of x: every matrix that reads h is one
+ * matrix here, and both outputs are one product. The input matrix has rows
+ *   q | k | gate | up,
+ * in that order, and its results go four ways: q as they are; k into row
+ * position % cache_rows of a ring of keys; sigmoid(gate); relu(up)^2. The
+ * output matrix has the columns of the attention output, then those of `up`. */
+struct FanOut {
+  int k_row, gate_row, up_row; /* where each part begins; multiples of 8 */
+  int cache_rows;
+  float *gate;                 /* [batch or positions][gate_stride] */
+  int64_t gate_stride;
+  float *up;
+  int64_t up_stride;
+};
+struct FanArgs {
+  const void *w;
+  int fmt; /* kFmtF32 or kFmtBf16 */
+  int rows, cols;
+  const float *x;
+  int64_t x_stride;
+  int batch;
+  const float *norm_w; /* NULL: x is normalised already */
+  int norm_n;
+  float eps;
+  float *q_out;
+  int64_t q_stride;
+  float *k_cache;
+  int64_t cache_batch_stride;
+  const int32_t *positions;
+  FanOut out;
+};
+const char *fan_proj(const FanArgs &a, cudaStream_t stream);
 
 /* The unfused pieces, for the operator surface. */
 const char *rope_and_store(float *q_out, float *k_cache, float *v_cache,
@@ -340,9 +375,20 @@ const char *rows_fp8_three_terms(void *out, const void *codes, const void *scale
                                  int n, int cols, cudaStream_t stream);
 const char *rows_spread_terms(void *out, const void *terms, int t, int cols,
                               int segments, const int *from, cudaStream_t stream);
-/* terms of RMSNorm(x[t]) * w for every position (nn_rms_norm_rows). */
-const char *rows_norm_terms(void *terms, const float *x, const void *w, int t,
-                            int dim, float eps, cudaStream_t stream);
+/* The gains of an RMSNorm: bf16 values, or f32 ones; n: how many values of a
+   row its mean is over, when rows end in zeros that only fill them up (0: all). */
+struct NormGain {
+  const void *gain;
+  bool f32;
+  int n;
+  NormGain(const void *bf16_gain) : gain(bf16_gain), f32(false), n(0) {}
+  NormGain(const float *f32_gain, int count) : gain(f32_gain), f32(true), n(count) {}
+};
+/* terms of RMSNorm(x[t]) * w for every position (nn_rms_norm_rows), or, with
+   `pick` (device memory), of the t positions it lists. */
+const char *rows_norm_terms(void *terms, const float *x, NormGain w, int t, int dim,
+                            float eps, cudaStream_t stream,
+                            const int32_t *pick = nullptr);
 /* bias + half-split RoPE; q to q_out [t][q_heads*hd], k and v to cache rows
    first_pos[0] + t. */
 const char *rows_qkv_finish(const float *partials, int splits, int t, int q_heads,
@@ -357,7 +403,7 @@ const char *rows_residual_finish(float *x, const float *partials, int splits, in
 /* x[t] += the product, then the terms of RMSNorm(x[t]) * w: the residual add
    and the normalisation that follows it, in one pass (dim <= 8192). */
 const char *rows_residual_norm(void *terms, float *x, const float *partials,
-                               int splits, int t, const void *w, int dim, float eps,
+                               int splits, int t, NormGain w, int dim, float eps,
                                cudaStream_t stream);
 const char *rows_swiglu_finish(void *terms, const float *partials, int splits, int t,
                                int hidden, cudaStream_t stream);
@@ -367,6 +413,67 @@ const char *rows_attention(void *terms, const float *q, const float *k_cache,
                            const float *v_cache, const int32_t *first_pos, int t,
                            int q_heads, int kv_heads, int hd, cudaStream_t stream);
 int rows_status();
+
+/* ---- what a parallel block needs besides (parallel_block.cu, window_attention.cu)
+ * Token rows into the residual: scale * table[token], plus the sinusoid of the
+ * position (sin at 2i, cos at 2i + 1; turns[i], f64: how much of a full turn the
+ * pair's angle advances per position), through an RMSNorm. Rows are `dim`
+ * values of which `width` are the model's and the rest zeros. per_sequence:
+ * row b is sequence b at positions[b]; else row t is at positions[0] + t. A token
+ * outside the table gives a row of NaN. */
+struct PositionEmbedArgs {
+  float *x;
+  const void *table;
+  bool table_bf16;
+  const int32_t *tokens;
+  int count, vocab, width, dim;
+  float scale;
+  const double *turns;
+  const float *gain;
+  float eps;
+  const int32_t *positions;
+  bool per_sequence;
+};
+const char *position_embed(const PositionEmbedArgs &a, cudaStream_t stream);
+
+/* Attention over the last `window` positions of a ring of keys that are the
+   values too (position t in row t % cache_rows), its output times `gate` element
+   by element. Scores without rotation. head_dim: a multiple of 4, at most
+   512; the row of a position is [kv_heads][head_dim]. */
+struct WindowAttnArgs {
+  const float *q;   /* [batch or positions][q_stride] */
+  int64_t q_stride;
+  const float *cache;
+  int64_t cache_batch_stride;
+  int cache_rows, window;
+  float scale;
+  const float *gate; /* [batch or positions][gate_stride] */
+  int64_t gate_stride;
+  int q_heads, kv_heads, head_dim;
+  const int32_t *positions; /* of each sequence; of the first of the positions */
+};
+/* One new token of each of `batch` sequences. cache_rows >= window. Rows below
+   the position were written before the chain of dependent launches began. */
+const char *window_attention_decode(const WindowAttnArgs &a, int batch, float *out,
+                                    int64_t out_stride, cudaStream_t stream);
+/* t positions of one sequence, whose own keys are in the ring (cache_rows >=
+   window - 1 + t); the output as terms, in the first columns of [t, 3 cols]. */
+const char *window_attention_rows(const WindowAttnArgs &a, int t, void *terms,
+                                  int cols, cudaStream_t stream);
+/* After the input GEMM: its results where fan_proj puts them, the ring's row
+   of position t being (positions[0] + t) % cache_rows, and relu(up)^2 as terms
+   in columns out_col.. of [t, 3 out_cols]. n rows of the matrix. */
+const char *rows_fan_finish(const float *partials, int splits, int t, int n,
+                            const FanOut &out, const int32_t *positions, float *q_out,
+                            int64_t q_stride, float *k_cache, void *terms, int out_cols,
+                            int out_col, cudaStream_t stream);
+/* partials[t][n] = W[n, cols] x[t, cols] on the FP32 pipe, for f32 W; x is the
+   sum of its three terms. One run. cols a multiple of 16. */
+const char *rows_gemm_f32(const void *terms, const float *w, int t, int n, int cols,
+                          float *partials, cudaStream_t stream);
+/* out[t][r] = the runs' sum, r below n. */
+const char *rows_sum(float *out, const float *partials, int splits, int t, int n,
+                     cudaStream_t stream);
 
 /* nn_top_k (nn.vx:904-938): ids[j] = the index of the j-th largest of the
    first n logits (n <= 256; of equal values the lower index first), weights[j]

@@ -38,6 +38,14 @@ __device__ __forceinline__ float warp_max(float v) {
   return v;
 }
 
+__device__ __forceinline__ float sigmoid(float v) {
+  return 1.0f / (1.0f + expf(0.0f - v));
+}
+__device__ __forceinline__ float squared_relu(float v) {
+  const float r = fmaxf(v, 0.0f);
+  return r * r;
+}
+
 /* The pushed exchange moves (value, call) pairs: an aligned 8-byte store
    arrives whole, so a pair that carries the expected call number is complete
    and is its own arrival flag. An item's two rows travel as two pairs in one
@@ -374,12 +382,14 @@ attention_unit(const AttnArgs &a, int split_idx, int y, int b, int warp,
   }
 }
 
+} // namespace
+
 /* ---------------------------------------------------------------- row dots
  * One kernel for every projection of the decoder.  An ITEM is a pair of weight
  * rows whose results the epilogue needs together; a warp owns a contiguous,
  * balanced range of items and streams both rows of an item at once. */
 enum { EPI_STORE = 0, EPI_ADD = 1, EPI_BIAS = 2, EPI_SWIGLU = 3, EPI_QKV = 4,
-       EPI_PUSH = 5 };
+       EPI_PUSH = 5, EPI_FAN = 6 };
 
 struct RowDotParams {
   /* weights */
@@ -423,7 +433,24 @@ struct RowDotParams {
   int64_t expert_bytes, scale_bytes;
   const float *add_scale;
   int scales_in_ring; /* Q4_0: set by the launcher */
+  /* values the mean square of the RMSNorm is taken over, when rows of x end in
+     zeros that only fill them up; 0: cols */
+  int norm_n;
+  /* EPI_FAN (see FanOut in kernels.h) */
+  FanOut fan;
 };
+
+/* The projection kernel by weight format (rowdot_f32.cu, rowdot_bf16.cu,
+   rowdot_quant.cu): epi is an EPI_* code, fmt kFmtFp8 or kFmtQ4. */
+const char *rowdot_f32(int epi, RowDotParams &p, cudaStream_t stream);
+const char *rowdot_bf16(int epi, RowDotParams &p, cudaStream_t stream);
+const char *rowdot_quant(int epi, RowDotParams &p, int fmt, cudaStream_t stream);
+int rowdot_f32_status();
+int rowdot_bf16_status();
+int rowdot_quant_status();
+
+
+namespace {
 
 /* Weight formats. A row is a run of 16-byte words; a word holds E weights:
    4 f32, 8 bf16, 16 fp8 (f8e4m3 codes with an f32 scale per block of 128 x 128

@@ -1,0 +1,206 @@
+/* parallel_block.cu -- the small kernels around the two products of a parallel
+ * block, and the f32 product of a prompt's positions.
+ *
+ * A parallel block reads one norm of the residual in all its input matrices, so
+ * they are one matrix with rows q | k | gate | up, and adds the sum of its two
+ * outputs, so they are one matrix whose columns are the attention output's and
+ * then `up`'s.  A decode step is three launches a layer (fan_proj, window
+ * attention, matvec with a residual add), a prompt five (GEMM, rows_fan_finish,
+ * window attention, GEMM, residual add and norm).
+ */
+#include "kernels.h"
+#include "launch.cuh"
+#include "launch_util.h"
+#include "nn_device.cuh"
+#include "terms.cuh"
+
+#include <cstdio>
+
+namespace vxb {
+namespace {
+
+/* ---- token rows with their position, normalised: a block per row ------------- */
+__global__ void __launch_bounds__(256) position_embed_kernel(const PositionEmbedArgs a) {
+  __shared__ float red[8];
+  chain_release();
+  chain_wait();
+  const int64_t t = blockIdx.x;
+  const int token = a.tokens[t];
+  const int pos = a.per_sequence ? a.positions[t] : a.positions[0] + (int)t;
+  float *row = a.x + t * a.dim;
+  if (token < 0 || token >= a.vocab) {
+    for (int i = threadIdx.x; i < a.dim; i += blockDim.x)
+      row[i] = i < a.width ? __int_as_float(0x7fc00000) : 0.0f;
+    return;
+  }
+  float ss = 0.0f;
+  for (int i = threadIdx.x; i < a.width; i += blockDim.x) {
+    const int64_t at = (int64_t)token * a.dim + i;
+    const float e = a.table_bf16 ? bf16_val(a.table, at) : ((const float *)a.table)[at];
+    /* the angle in turns: what is left of it after whole turns is exact enough
+       in f64 for any position, and small in f32 */
+    const double turns = pos * a.turns[i / 2];
+    const float half_turns = 2.0f * (float)(turns - rint(turns));
+    const float p = i % 2 == 0 ? sinpif(half_turns) : cospif(half_turns);
+    const float v = fmaf(e, a.scale, p);
+    row[i] = v;
+    ss = fmaf(v, v, ss);
+  }
+  ss = warp_sum(ss);
+  if ((threadIdx.x & 31) == 0)
+    red[threadIdx.x >> 5] = ss;
+  __syncthreads();
+  float total = 0.0f;
+  for (int k = 0; k < 8; ++k) /* fixed order */
+    total += red[k];
+  const float inv = 1.0f / sqrtf(total / (float)a.width + a.eps);
+  for (int i = threadIdx.x; i < a.dim; i += blockDim.x) /* its own values again */
+    row[i] = i < a.width ? row[i] * inv * a.gain[i] : 0.0f;
+}
+
+/* ---- after the input GEMM: a thread per (position, eight rows) ---------------- */
+__global__ void __launch_bounds__(256)
+fan_finish_kernel(const float *partials, int splits, int t_count, int n,
+                  const FanOut f, const int32_t *positions, float *q_out,
+                  int64_t q_stride, float *k_cache, __nv_bfloat16 *terms, int out_cols,
+                  int out_col) {
+  chain_release();
+  chain_wait();
+  const int per_row = n / 8;
+  const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= (int64_t)t_count * per_row)
+    return;
+  const int64_t t = idx / per_row;
+  const int r = (int)(idx - t * per_row) * 8;
+  const float4 lo = sum_runs4(partials, splits, t_count, n, t, r);
+  const float4 hi = sum_runs4(partials, splits, t_count, n, t, r + 4);
+  float v[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+  float *dst;
+  if (r < f.k_row) {
+    dst = q_out + t * q_stride + r;
+  } else if (r < f.gate_row) {
+    const int row = (positions[0] + (int)t) % f.cache_rows;
+    dst = k_cache + (int64_t)row * (f.gate_row - f.k_row) + r - f.k_row;
+  } else if (r < f.up_row) {
+#pragma unroll
+    for (int e = 0; e < 8; ++e)
+      v[e] = sigmoid(v[e]);
+    dst = f.gate + t * f.gate_stride + r - f.gate_row;
+  } else {
+#pragma unroll
+    for (int e = 0; e < 8; ++e)
+      v[e] = squared_relu(v[e]);
+    store_terms8(terms, out_cols, t, out_col + r - f.up_row, v);
+    return;
+  }
+  *reinterpret_cast<float4 *>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+  *reinterpret_cast<float4 *>(dst + 4) = make_float4(v[4], v[5], v[6], v[7]);
+}
+
+__global__ void __launch_bounds__(256)
+sum_kernel(float *out, const float *partials, int splits, int t_count, int n) {
+  chain_release();
+  chain_wait();
+  const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= (int64_t)t_count * n)
+    return;
+  const int64_t t = idx / n;
+  out[idx] = sum_runs(partials, splits, t_count, n, t, idx - t * n);
+}
+
+/* ---- the f32 product on the FP32 pipe: 64 positions x 64 rows a block, 4 x 4 a
+   thread, the terms added up again (exactly) on their way into shared memory --- */
+constexpr int GT = 64, GC = 16;
+__global__ void __launch_bounds__(256)
+rows_gemm_f32_kernel(const __nv_bfloat16 *terms, const float *w, int t_count, int n,
+                     int cols, float *out) {
+  __shared__ __align__(16) float sx[GC][GT + 4], sw[GC][GT + 4];
+  chain_release();
+  chain_wait();
+  const int tid = threadIdx.x, ty = tid / 16, tx = tid % 16;
+  const int t0 = blockIdx.y * GT, n0 = blockIdx.x * GT;
+  /* a thread stages four columns of one position and of one matrix row */
+  const int lr = tid / 4, lc = tid % 4 * 4;
+  float acc[4][4] = {};
+  for (int c0 = 0; c0 < cols; c0 += GC) {
+    float xv[4] = {0, 0, 0, 0}, wv[4] = {0, 0, 0, 0};
+    if (t0 + lr < t_count) {
+      const __nv_bfloat16 *row = terms + (int64_t)(t0 + lr) * 3 * cols + c0 + lc;
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        xv[e] = (bf16_val(row, e) + bf16_val(row, cols + e)) +
+                bf16_val(row, 2 * (int64_t)cols + e);
+    }
+    if (n0 + lr < n) {
+      const float4 v =
+          *reinterpret_cast<const float4 *>(w + (int64_t)(n0 + lr) * cols + c0 + lc);
+      wv[0] = v.x; wv[1] = v.y; wv[2] = v.z; wv[3] = v.w;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      sx[lc + e][lr] = xv[e];
+      sw[lc + e][lr] = wv[e];
+    }
+    __syncthreads();
+#pragma unroll
+    for (int c = 0; c < GC; ++c) {
+      const float4 xa = *reinterpret_cast<const float4 *>(&sx[c][ty * 4]);
+      const float4 wa = *reinterpret_cast<const float4 *>(&sw[c][tx * 4]);
+      const float xs[4] = {xa.x, xa.y, xa.z, xa.w}, ws[4] = {wa.x, wa.y, wa.z, wa.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i)
+#pragma unroll
+        for (int j = 0; j < 4; ++j)
+          acc[i][j] = fmaf(xs[i], ws[j], acc[i][j]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+      if (t0 + ty * 4 + i < t_count && n0 + tx * 4 + j < n)
+        out[(int64_t)(t0 + ty * 4 + i) * n + n0 + tx * 4 + j] = acc[i][j];
+}
+
+} // namespace
+
+const char *position_embed(const PositionEmbedArgs &a, cudaStream_t stream) {
+  if (a.count <= 0)
+    return nullptr;
+  launch_chained(position_embed_kernel, dim3(a.count), dim3(256), 0, stream, a);
+  return check_launch("the embedding launch");
+}
+
+const char *rows_fan_finish(const float *partials, int splits, int t, int n,
+                            const FanOut &out, const int32_t *positions, float *q_out,
+                            int64_t q_stride, float *k_cache, void *terms, int out_cols,
+                            int out_col, cudaStream_t stream) {
+  if ((n | out.k_row | out.gate_row | out.up_row | out_cols | out_col) % 8 != 0)
+    return "the parts of an input projection are multiples of 8 rows";
+  const int64_t count = (int64_t)t * (n / 8);
+  launch_chained(fan_finish_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0,
+                 stream, partials, splits, t, n, out, positions, q_out, q_stride,
+                 k_cache, (__nv_bfloat16 *)terms, out_cols, out_col);
+  return check_launch("the parts of an input projection");
+}
+
+const char *rows_sum(float *out, const float *partials, int splits, int t, int n,
+                     cudaStream_t stream) {
+  const int64_t count = (int64_t)t * n;
+  launch_chained(sum_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0, stream,
+                 out, partials, splits, t, n);
+  return check_launch("the sum of a product's runs");
+}
+
+const char *rows_gemm_f32(const void *terms, const float *w, int t, int n, int cols,
+                          float *partials, cudaStream_t stream) {
+  if (cols % GC != 0 || ((uintptr_t)w & 15))
+    return "the f32 product of many positions takes columns in multiples of 16";
+  launch_chained(rows_gemm_f32_kernel, dim3((n + GT - 1) / GT, (t + GT - 1) / GT),
+                 dim3(256), 0, stream, (const __nv_bfloat16 *)terms, w, t, n, cols,
+                 partials);
+  return check_launch("the f32 product of many positions");
+}
+
+} // namespace vxb

@@ -31,6 +31,7 @@
 #include "kernels.h"
 #include "launch.cuh"
 #include "ptx.cuh"
+#include "terms.cuh"
 
 #include <cuda_bf16.h>
 
@@ -257,83 +258,21 @@ rows_gemm_kernel(const __grid_constant__ CUtensorMap map_x,
 }
 
 /* ---- what sits between the GEMMs ------------------------------------------- */
-__device__ __forceinline__ float bf16_val(const void *p, int64_t i) {
-  return __uint_as_float((uint32_t)((const uint16_t *)p)[i] << 16);
-}
-/* v as three bf16 terms at column i of row t of a [T, 3 cols] matrix. */
-__device__ __forceinline__ void store_terms(__nv_bfloat16 *terms, int cols,
-                                            int64_t t, int i, float v) {
-  const __nv_bfloat16 t1 = __float2bfloat16(v);
-  const float r1 = v - __bfloat162float(t1);
-  const __nv_bfloat16 t2 = __float2bfloat16(r1);
-  const float r2 = r1 - __bfloat162float(t2);
-  __nv_bfloat16 *row = terms + t * 3 * cols;
-  row[i] = t1;
-  row[cols + i] = t2;
-  row[2 * cols + i] = __float2bfloat16(r2);
-}
-/* The sum of the runs' partials of (t, r), in run order. */
-__device__ __forceinline__ float sum_runs(const float *partials, int splits,
-                                          int64_t t_count, int64_t n, int64_t t,
-                                          int64_t r) {
-  float s = partials[t * n + r];
-  for (int k = 1; k < splits; ++k)
-    s += partials[((int64_t)k * t_count + t) * n + r];
-  return s;
-}
-
-/* The same for four consecutive values (r a multiple of 4). */
-__device__ __forceinline__ float4 sum_runs4(const float *partials, int splits,
-                                            int64_t t_count, int64_t n, int64_t t,
-                                            int64_t r) {
-  float4 s = *reinterpret_cast<const float4 *>(partials + t * n + r);
-  for (int k = 1; k < splits; ++k) {
-    const float4 v = *reinterpret_cast<const float4 *>(
-        partials + ((int64_t)k * t_count + t) * n + r);
-    s.x += v.x; s.y += v.y; s.z += v.z; s.w += v.w;
-  }
-  return s;
-}
-/* Eight consecutive values (i a multiple of 8) as their three terms: one
-   16-byte store per term. */
-__device__ __forceinline__ void store_terms8(__nv_bfloat16 *terms, int cols,
-                                             int64_t t, int i, const float (&v)[8]) {
-  uint32_t w1[4], w2[4], w3[4];
-#pragma unroll
-  for (int j = 0; j < 4; ++j) {
-    uint32_t parts[3] = {0, 0, 0};
-#pragma unroll
-    for (int h = 0; h < 2; ++h) {
-      const float x = v[2 * j + h];
-      const __nv_bfloat16 t1 = __float2bfloat16(x);
-      const float r1 = x - __bfloat162float(t1);
-      const __nv_bfloat16 t2 = __float2bfloat16(r1);
-      const float r2 = r1 - __bfloat162float(t2);
-      const __nv_bfloat16 t3 = __float2bfloat16(r2);
-      parts[0] |= (uint32_t)__bfloat16_as_ushort(t1) << (16 * h);
-      parts[1] |= (uint32_t)__bfloat16_as_ushort(t2) << (16 * h);
-      parts[2] |= (uint32_t)__bfloat16_as_ushort(t3) << (16 * h);
-    }
-    w1[j] = parts[0];
-    w2[j] = parts[1];
-    w3[j] = parts[2];
-  }
-  __nv_bfloat16 *row = terms + t * 3 * cols;
-  *reinterpret_cast<uint4 *>(row + i) = make_uint4(w1[0], w1[1], w1[2], w1[3]);
-  *reinterpret_cast<uint4 *>(row + cols + i) = make_uint4(w2[0], w2[1], w2[2], w2[3]);
-  *reinterpret_cast<uint4 *>(row + 2 * cols + i) = make_uint4(w3[0], w3[1], w3[2], w3[3]);
+/* The gains of a norm are bf16, or f32 where they are not a bf16 value (1 + w). */
+__device__ __forceinline__ float gain_at(const NormGain &w, int i) {
+  return w.f32 ? ((const float *)w.gain)[i] : bf16_val(w.gain, i);
 }
 
 /* nn_rms_norm_rows (nn.vx:2835): terms of x[t] / sqrt(mean(x[t]^2) + eps) * w;
-   one block per position. */
+   one block per position. pick: the positions, block by block (NULL: all). */
 __global__ void __launch_bounds__(256)
-norm_terms_kernel(__nv_bfloat16 *terms, const float *x, const void *w, int dim,
-                  float eps) {
+norm_terms_kernel(__nv_bfloat16 *terms, const float *x, const NormGain w, int dim,
+                  float eps, const int32_t *pick) {
   __shared__ float red[8];
   chain_release();
   chain_wait();
   const int64_t t = blockIdx.x;
-  const float *xr = x + t * dim;
+  const float *xr = x + (pick ? pick[t] : t) * (int64_t)dim;
   float ss = 0.0f;
   for (int i = threadIdx.x; i < dim; i += blockDim.x)
     ss = fmaf(xr[i], xr[i], ss);
@@ -345,9 +284,9 @@ norm_terms_kernel(__nv_bfloat16 *terms, const float *x, const void *w, int dim,
   float total = 0.0f;
   for (int k = 0; k < 8; ++k) /* fixed order */
     total += red[k];
-  const float inv = 1.0f / sqrtf(total / (float)dim + eps);
+  const float inv = 1.0f / sqrtf(total / (float)(w.n ? w.n : dim) + eps);
   for (int i = threadIdx.x; i < dim; i += blockDim.x)
-    store_terms(terms, dim, t, i, xr[i] * bf16_val(w, i) * inv);
+    store_terms(terms, dim, t, i, xr[i] * gain_at(w, i) * inv);
 }
 
 /* After the output or the down projection, when an RMSNorm follows: x[t] += the
@@ -356,7 +295,7 @@ norm_terms_kernel(__nv_bfloat16 *terms, const float *x, const void *w, int dim,
    norm_terms_kernel). One block per position; dim <= 256 * 32. */
 __global__ void __launch_bounds__(256)
 residual_norm_kernel(__nv_bfloat16 *terms, float *x, const float *partials,
-                     int splits, int t_count, const void *w, int dim, float eps) {
+                     int splits, int t_count, const NormGain w, int dim, float eps) {
   __shared__ float red[8];
   chain_release();
   chain_wait();
@@ -383,12 +322,12 @@ residual_norm_kernel(__nv_bfloat16 *terms, float *x, const float *partials,
   float total = 0.0f;
   for (int k = 0; k < 8; ++k) /* fixed order */
     total += red[k];
-  const float inv = 1.0f / sqrtf(total / (float)dim + eps);
+  const float inv = 1.0f / sqrtf(total / (float)(w.n ? w.n : dim) + eps);
 #pragma unroll
   for (int k = 0; k < PER; ++k) {
     const int i = threadIdx.x + k * 256;
     if (i < dim)
-      store_terms(terms, dim, t, i, v[k] * bf16_val(w, i) * inv);
+      store_terms(terms, dim, t, i, v[k] * gain_at(w, i) * inv);
   }
 }
 
@@ -886,10 +825,10 @@ const char *rows_spread_terms(void *out, const void *terms, int t, int cols,
   return last_launch("the spread terms");
 }
 
-const char *rows_norm_terms(void *terms, const float *x, const void *w, int t,
-                            int dim, float eps, cudaStream_t stream) {
+const char *rows_norm_terms(void *terms, const float *x, NormGain w, int t, int dim,
+                            float eps, cudaStream_t stream, const int32_t *pick) {
   launch_chained(norm_terms_kernel, dim3(t), dim3(256), 0, stream,
-                 (__nv_bfloat16 *)terms, x, w, dim, eps);
+                 (__nv_bfloat16 *)terms, x, w, dim, eps, pick);
   return last_launch("the multi-position RMSNorm");
 }
 
@@ -916,7 +855,7 @@ const char *rows_residual_finish(float *x, const float *partials, int splits, in
 }
 
 const char *rows_residual_norm(void *terms, float *x, const float *partials,
-                               int splits, int t, const void *w, int dim, float eps,
+                               int splits, int t, NormGain w, int dim, float eps,
                                cudaStream_t stream) {
   if (dim > 256 * 32)
     return "the fused residual and RMSNorm take rows of at most 8192 values";

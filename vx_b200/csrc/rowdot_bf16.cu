@@ -1,0 +1,21 @@
+/* rowdot_bf16.cu -- the projection kernel with bf16 weights, every epilogue. */
+#include "rowdot.cuh"
+
+namespace vxb {
+
+const char *rowdot_bf16(int epi, RowDotParams &p, cudaStream_t stream) {
+  switch (epi) {
+  case EPI_STORE: return launch_rowdot_w<__nv_bfloat16, EPI_STORE>(p, stream);
+  case EPI_ADD: return launch_rowdot_w<__nv_bfloat16, EPI_ADD>(p, stream);
+  case EPI_BIAS: return launch_rowdot_w<__nv_bfloat16, EPI_BIAS>(p, stream);
+  case EPI_SWIGLU: return launch_rowdot_w<__nv_bfloat16, EPI_SWIGLU>(p, stream);
+  case EPI_QKV: return launch_rowdot_w<__nv_bfloat16, EPI_QKV>(p, stream);
+  case EPI_PUSH: return launch_rowdot_w<__nv_bfloat16, EPI_PUSH>(p, stream);
+  case EPI_FAN: return launch_rowdot_w<__nv_bfloat16, EPI_FAN>(p, stream);
+  default: return "unknown epilogue";
+  }
+}
+
+int rowdot_bf16_status() { return take_rowdot_status(); }
+
+} // namespace vxb

@@ -1,6 +1,6 @@
 /* rowdot_quant_mma.cuh -- the fp8 and Q4_0 projections of ONE sequence on the
  * tensor cores (nn_matvec_fp8 / nn_swiglu_fp8 / nn_qkv_fp8, nn.vx:1306-1577;
- * the Q4_0 forms, nn.vx:1666-2190). Part of nn_kernels.cu (included there).
+ * the Q4_0 forms, nn.vx:1666-2190). Part of rowdot_quant.cu (included there).
  *
  * With one-byte and half-byte weights the projection kernel is bound by
  * instruction issue, not by HBM: every weight costs a conversion to f32, a

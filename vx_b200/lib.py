@@ -46,6 +46,8 @@ EXTRA_SYMBOLS = [
     "vx_nn_moe_down_q4_add",
     "vx_decoder_create", "vx_decoder_destroy", "vx_decoder_reset",
     "vx_decoder_step", "vx_decoder_prefill", "vx_decoder_logits",
+    "vx_decoder_logits_pitch", "vx_decoder_create_parallel",
+    "vx_decoder_prefill_logits",
     "vx_decoder_kernels_per_step",
     "vx_decoder_step_trace",
     "vx_decoder_kv_cache", "vx_decoder_kv_cache_bytes", "vx_decoder_adopt_kv",
@@ -79,6 +81,23 @@ class DecoderWeights(C.Structure):
                 ("cos", C.c_void_p), ("sin", C.c_void_p)] + \
                [(n, C.POINTER(C.c_void_p)) for n in
                 ("s_qkv", "s_o", "s_gate_up", "s_down")]
+
+
+class ParallelLayer(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in
+                ("q_heads", "kv_heads", "head_dim", "hidden", "window")] + \
+               [("score_scale", C.c_float)] + \
+               [(n, C.c_void_p) for n in ("norm", "w_in", "w_out")]
+
+
+class ParallelConfig(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in
+                ("width", "dim", "n_layers", "vocab", "vocab_rows", "max_seq",
+                 "weights_bf16", "batch", "prefill_rows")] + \
+               [("eps", C.c_float), ("embed_scale", C.c_float)] + \
+               [(n, C.c_void_p) for n in
+                ("embed", "classifier", "embed_norm", "final_norm", "turns")] + \
+               [("layers", C.POINTER(ParallelLayer))]
 
 
 class Llama2cConfig(C.Structure):
@@ -140,6 +159,12 @@ def lib():
     L.vx_decoder_step.argtypes = [vp, vp, vp]
     L.vx_decoder_prefill.restype = i32
     L.vx_decoder_prefill.argtypes = [vp, vp, i32]
+    L.vx_decoder_create_parallel.restype = vp
+    L.vx_decoder_create_parallel.argtypes = [C.POINTER(ParallelConfig)]
+    L.vx_decoder_prefill_logits.restype = i32
+    L.vx_decoder_prefill_logits.argtypes = [vp, vp, i32, vp, i32, vp]
+    L.vx_decoder_logits_pitch.restype = i32
+    L.vx_decoder_logits_pitch.argtypes = [vp]
     L.vx_decoder_logits.restype = vp
     L.vx_decoder_logits.argtypes = [vp]
     L.vx_decoder_kv_cache.restype = vp

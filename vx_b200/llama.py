@@ -14,7 +14,7 @@ import ctypes as C
 import numpy as np
 
 from . import abi
-from .lib import DecoderConfig, DecoderWeights, Llama2cConfig, lib
+from .lib import DecoderConfig, DecoderWeights, Llama2cConfig, ParallelConfig, lib
 
 
 def _ptr_array(ptrs):
@@ -46,6 +46,20 @@ class Decoder:
             max_seq=max_seq or head.seq_len, eps=1e-5, rope_theta=10000.0,
             weights_bf16=0, batch=batch, tp_ranks=1, tp_reduce=0)
         self.keep, self._arrays, self._w, self.handle = None, {}, None, handle
+        self._in = (C.c_int32 * 32)()
+        self._out = (C.c_int32 * 32)()
+        return self
+
+    @classmethod
+    def from_parallel(cls, cfg, keep=None):
+        """A decoder of parallel blocks (vx_decoder_create_parallel); cfg is a
+        ParallelConfig, `keep` holds whatever owns its memory."""
+        handle = lib().vx_decoder_create_parallel(C.byref(cfg))
+        if not handle:
+            raise ValueError(lib().vx_b200_last_error().decode())
+        self = cls.__new__(cls)
+        self.cfg, self.keep, self.handle = cfg, keep, handle
+        self._arrays, self._w = {}, None
         self._in = (C.c_int32 * 32)()
         self._out = (C.c_int32 * 32)()
         return self
@@ -98,14 +112,47 @@ class Decoder:
             self.step([t], fetch=False)
         return self.step([tokens[-1]])[0]
 
+    def feed(self, tokens, want=()):
+        """The next tokens of a one-sequence decoder, and the logits
+        [len(want), vocab] after those whose places are in `want` (ascending):
+        in one pass where the decoder has one that gives logits, single steps
+        otherwise."""
+        tokens, want = [int(t) for t in tokens], [int(w) for w in want]
+        if isinstance(self.cfg, ParallelConfig) and len(tokens) > 1:
+            arr = (C.c_int32 * len(tokens))(*tokens)
+            places = (C.c_int32 * max(len(want), 1))(*want)
+            out = np.empty((len(want), self.cfg.vocab), np.float32)
+            if lib().vx_decoder_prefill_logits(
+                    self.handle, arr, len(tokens), places, len(want),
+                    out.ctypes.data_as(C.c_void_p)) < 0:
+                raise ValueError(lib().vx_b200_last_error().decode())
+            return out
+        rows = []
+        for i, t in enumerate(tokens):
+            asked = i in want
+            self.step([t], fetch=asked)
+            if asked:
+                rows.append(self.logits()[0])
+        return np.array(rows, np.float32).reshape(
+            (len(want), -1) if want else (0, self.cfg.vocab))
+
+    def generate(self, prompt, count):
+        """`count` greedy tokens after a prompt of a one-sequence decoder; each
+        goes from one step to the next without leaving the GPU."""
+        tokens = [self.prefill(prompt)]
+        while len(tokens) < count:
+            tokens.append(self.step()[0])
+        return tokens[:count]
+
     def logits(self):
         """[batch, local vocab] f32 from the last step."""
-        n = self.cfg.batch * (self.cfg.vocab // max(self.cfg.tp_ranks, 1))
-        out = np.empty(n, np.float32)
+        pitch = lib().vx_decoder_logits_pitch(self.handle)
+        out = np.empty((self.cfg.batch, pitch), np.float32)
         lib().vx_plugin_transfer_device_to_host(
             lib().vx_decoder_logits(self.handle),
             out.ctypes.data_as(C.c_void_p), out.nbytes, abi.home_gpu())
-        return out.reshape(self.cfg.batch, -1)
+        vocab = self.cfg.vocab // max(getattr(self.cfg, "tp_ranks", 1), 1)
+        return np.ascontiguousarray(out[:, :vocab])
 
     @property
     def stream(self):
