@@ -295,7 +295,7 @@ int32_t vx_decoder_logits_pitch(const vx_decoder *d);
    [layer][sequence][max_seq][kv_heads][head_dim], vx_decoder_kv_cache_bytes()
    bytes each. What a prefill process hands to a decode process
    (handoff_kv, tests/backend/pass/llama2.vx:431-458: the caches travel by
-   vx_plugin_transfer_peer). */
+   vx_plugin_transfer_peer). Waits for the steps queued so far, which write it. */
 float *vx_decoder_kv_cache(vx_decoder *d, int32_t which);
 int64_t vx_decoder_kv_cache_bytes(const vx_decoder *d);
 /* The receiving side of that hand-off: copies rows 0 .. positions-1 of every

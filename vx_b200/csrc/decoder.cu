@@ -1275,6 +1275,7 @@ vx_decoder *vx_decoder_from_llama2c(const char *path, int32_t batch,
 const float *vx_decoder_logits(const vx_decoder *d) { return d->logits; }
 
 float *vx_decoder_kv_cache(vx_decoder *d, int32_t which) {
+  CUDA_OK(cudaStreamSynchronize(d->stream)); /* queued steps still write it */
   return which == 0 ? d->k_cache : which == 1 ? d->v_cache : nullptr;
 }
 

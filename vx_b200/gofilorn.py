@@ -77,13 +77,14 @@ class GofilornConfig:
             layers.append(LayerShape(m["heads"], m["kv_heads"], m["dim"],
                                      m["mask"]["size"], m["scale"],
                                      mlp["ff"] if mlp is not None else 0, source))
+        named = [layer.source for layer in layers]
         for i, layer in enumerate(layers):
             for _ in layers:        # to the layer that has tensors of its own
-                layer.source = layers[layer.source].source
-            owner = layers[layer.source]
-            if owner.source != layer.source or not layer.same_tensors(owner):
+                layer.source = named[layer.source]
+            if named[layer.source] != layer.source or \
+                    not layer.same_tensors(layers[layer.source]):
                 raise ValueError("layer %d cannot use the tensors of layer %d"
-                                 % (i, layer.source))
+                                 % (i, named[i]))
         return cls(config["width"], config["vocab"], config["norm"]["eps"],
                    config["embedding"]["scale"], layers)
 
