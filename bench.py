@@ -11,6 +11,7 @@ sequences per step), each with its error against the CPU oracle on sampled
 rows, the roofline of the dominant kernel, and the CPU baseline.
 
   python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
+  python bench.py --design gofilorn      another design beside the Llama decoder
 """
 import argparse
 import ctypes as C
@@ -915,6 +916,105 @@ def run_ours(args):
         dist.destroy_process_group()
 
 
+# ---- another design beside the Llama decoder of equal size -------------------------
+# Layers like a real model's, in two widths; the Llama decoder beside each has the
+# same width, heads and number of weights a layer within 1 % (one key head as well).
+DESIGN_SIZES = {
+    "width2048": dict(width=2048, heads=16, ff=7424, window=1024, layers=16,
+                      llama_hidden=5632),
+    "width4096": dict(width=4096, heads=32, ff=14720, window=1024, layers=8,
+                      llama_hidden=11008),
+}
+DESIGN_VOCAB, DESIGN_PROMPTS = 32000, (512, 2048)
+
+
+def gofilorn_of_size(s):
+    """(decoder, bytes of weights a step streams) of random weights."""
+    from vx_b200 import gofilorn
+    entry = dict(type="attention", mlp=dict(kind="dense", ff=s["ff"]),
+                 mixer=dict(heads=s["heads"], kv_heads=1, dim=128, vdim=128,
+                            mask=dict(size=s["window"]), scale=128 ** -0.5))
+    cfg = gofilorn.GofilornConfig.from_dict(dict(
+        architecture="Gofilorn", width=s["width"], vocab=DESIGN_VOCAB,
+        embedding=dict(scale=1.0), norm=dict(eps=1e-5), layers=[entry] * s["layers"]))
+    weights = sum((l.in_rows + l.out_cols) * cfg.dim for l in cfg.layers)
+    return gofilorn.synthetic(cfg, MAX_SEQ), 2 * (weights + DESIGN_VOCAB * cfg.dim)
+
+
+def llama_of_size(s):
+    from vx_b200 import llama
+    shape = dict(dim=s["width"], hidden=s["llama_hidden"], n_layers=s["layers"],
+                 q_heads=s["heads"], kv_heads=1, head_dim=128, vocab=DESIGN_VOCAB)
+    return (llama.nn_bf16_model(max_seq=MAX_SEQ, **shape)[0],
+            llama.weight_bytes_per_token(**shape))
+
+
+def time_decoder(torch, dec, peaks, weight_bytes, steps, warmup):
+    """Prompt passes of several lengths and decoding after the first of them."""
+    from vx_b200.lib import lib
+    stream = torch.cuda.ExternalStream(dec.stream)
+    tokens = np.random.default_rng(8).integers(0, DESIGN_VOCAB, max(DESIGN_PROMPTS))
+    arr = (C.c_int32 * len(tokens))(*[int(t) for t in tokens])
+    out = {}
+    for n in DESIGN_PROMPTS:
+        times = []
+        for i in range(3 + 5):           # the median of five after three untimed ones
+            dec.reset()
+            ms = event_ms(torch, stream,
+                          lambda: lib().vx_decoder_prefill(dec.handle, arr, n))
+            if i >= 3:
+                times.append(ms)
+        ms = float(np.median(times))
+        # every weight of the layers meets every position once (the classifier none)
+        flop = (weight_bytes - 2 * DESIGN_VOCAB * dec.cfg.dim) * n
+        out["prefill_%d" % n] = dict(ms=ms, tokens_per_s=1e3 * n / ms,
+                                     tflops_of_weights=flop / ms / 1e9)
+    dec.reset()
+    lib().vx_decoder_prefill(dec.handle, arr, DESIGN_PROMPTS[0])
+    dec.step([1], fetch=False)
+    for _ in range(warmup):
+        dec.step(None, fetch=False)
+    torch.cuda.synchronize()
+    ms = event_ms(torch, stream, lambda: [dec.step(None, fetch=False)
+                                          for _ in range(steps)]) / steps
+    gbs = weight_bytes / ms / 1e6
+    out["decode"] = dict(ms_per_step=ms, tokens_per_s=1e3 / ms,
+                         weight_gbs=gbs, frac_of_measured_hbm=gbs / peaks["hbm_gbs"],
+                         kernels_per_step=dec.kernels_per_step)
+    return out
+
+
+def run_design(args):
+    """--design gofilorn: prefill and decode of the design at a few sizes, random
+    weights, one sequence, with the Llama decoder of equal size beside it."""
+    import torch
+    from vx_b200 import ops
+    peaks = measured_peaks()
+    sizes = {}
+    with ClockSampler(0) as clocks:
+        for name, s in DESIGN_SIZES.items():
+            if args.design_size and name != args.design_size:
+                continue
+            row = dict(size=s)
+            for which, make in (("gofilorn", gofilorn_of_size), ("llama", llama_of_size)):
+                if args.design_only and which != args.design_only:
+                    continue
+                dec, weight_bytes = make(s)
+                row[which] = time_decoder(torch, dec, peaks, weight_bytes, args.steps,
+                                          args.warmup)
+                row[which]["weight_mb"] = weight_bytes / 1e6
+                dec.close()
+                del dec
+                torch.cuda.empty_cache()
+            sizes[name] = row
+    print(json.dumps(dict(
+        metric="gofilorn_beside_llama", unit="tokens/s", steps=args.steps,
+        warmup=args.warmup, dtype="bf16 weights, f32 activations and accumulate",
+        data="synthetic", higher_is_better=True, sizes=sizes,
+        kernel_status=ops.kernel_status(), peaks=peaks, clocks=clocks.summary(),
+        l2_policy="a pass streams more weights than the 126 MB L2 holds")))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -923,9 +1023,19 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--no-extras", action="store_true",
                     help="skip the GEMM, flash-attention and batch-16 figures")
+    ap.add_argument("--design", choices=["gofilorn"],
+                    help="time this design beside the Llama decoder of equal size "
+                         "instead of the headline workload")
+    ap.add_argument("--design-size", choices=sorted(DESIGN_SIZES),
+                    help="with --design: this size only")
+    ap.add_argument("--design-only", choices=["gofilorn", "llama"],
+                    help="with --design: this decoder only")
     args = ap.parse_args()
     if args.warmup < 3:
         args.warmup = 3
+    if args.design:
+        run_design(args)
+        return
     if args.impl == "reference":
         run_reference(args)
     else:

@@ -57,6 +57,22 @@ def test_ctypes_can_bind_every_symbol(built):
         assert getattr(L, name)
 
 
+def test_the_smaller_library_has_every_entry_point(built):
+    """The library that serves decoders of parallel blocks only: the same exports,
+    with refusals in place of the kernels it leaves out."""
+    from vx_b200 import build
+    assert build.for_parallel_decoders() == build.LIB     # the whole one is there
+    small = build._library(build.PARALLEL_LIB, build.PARALLEL_SOURCES)
+    c_names = lambda path: {n for n in exported(path) if not n.startswith("_Z")}
+    assert c_names(small) == c_names(built)
+    r = run_child("from vx_b200.lib import lib, use\n"
+                  "use(%r)\n"
+                  "assert lib().vx_b200_gemm_q4(None, None, None, None, 1, 8, 32) == -1\n"
+                  "assert b'not part of this library' in lib().vx_b200_last_error()\n"
+                  % small)
+    assert r.returncode == 0, r.stderr
+
+
 def run_child(code):
     return subprocess.run([sys.executable, "-c", code], capture_output=True,
                           text=True, cwd=ROOT, timeout=120)

@@ -1,11 +1,16 @@
 """Build vx_b200/libvx_cuda_dispatch.so from csrc/*.cu with nvcc for sm_100a.
 
+for_parallel_decoders() gives a library that can serve decoders of parallel blocks:
+the whole one where it is built and up to date, else a smaller one of the same
+objects, libvx_parallel_decoder.so, which takes less compiling.
+
 The library is built in-tree, so that it travels with the source directory; it
 links the CUDA runtime statically and opens libcuda.so.1 and libnccl.so.2 at
 run time, so it loads (and answers symbol queries) on a machine with no GPU.
 """
 import concurrent.futures
 import os
+import shutil
 import subprocess
 import sys
 
@@ -14,11 +19,22 @@ ROOT = os.path.dirname(HERE)
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "_obj")
 LIB = os.path.join(HERE, "libvx_cuda_dispatch.so")
+PARALLEL_LIB = os.path.join(HERE, "libvx_parallel_decoder.so")
+NVCC = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
 
-SOURCES = ["rowdot_quant.cu", "rowdot_bf16.cu", "rowdot_f32.cu", "dispatch.cu", "gemm_simt.cu", "gemm_umma.cu", "gemm_umma_pair.cu", "nn_kernels.cu",
-           "nn_api.cu", "decoder.cu", "decoder_parallel.cu", "flash_attn.cu", "flash_attn_v2.cu", "static_scratch.cu", "rowdot_umma.cu", "prefill.cu", "quantize.cu", "step_kernel.cu", "gemm_f32_split.cu",
-           "moe_group.cu", "moe_grouped.cu", "gemm_fp8_rows.cu",
-           "window_attention.cu", "parallel_block.cu"]
+SOURCES = ["rowdot_quant.cu", "rowdot_bf16.cu", "rowdot_f32.cu", "nn_kernels.cu",
+           "dispatch.cu", "gemm_simt.cu", "gemm_umma.cu", "gemm_umma_pair.cu",
+           "nn_api.cu", "decoder.cu", "decoder_parallel.cu", "flash_attn.cu",
+           "flash_attn_v2.cu", "static_scratch.cu", "rowdot_umma.cu", "prefill.cu",
+           "quantize.cu", "step_kernel.cu", "gemm_f32_split.cu", "moe_group.cu",
+           "moe_grouped.cu", "gemm_fp8_rows.cu", "window_attention.cu",
+           "parallel_block.cu", "tensor_map.cu"]
+# what a decoder of parallel blocks runs and loads its weights with; absent.cu
+# stands for the rest
+PARALLEL_SOURCES = ["rowdot_bf16.cu", "rowdot_f32.cu", "nn_kernels.cu", "dispatch.cu",
+                    "nn_api.cu", "decoder.cu", "decoder_parallel.cu", "prefill.cu",
+                    "window_attention.cu", "parallel_block.cu", "tensor_map.cu",
+                    "absent.cu"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3",
               "-std=c++17", "-Xcompiler", "-fPIC", "-Xcompiler", "-Wall",
               "-I" + os.path.join(ROOT, "include"),
@@ -45,7 +61,7 @@ def _compile(src, verbose):
     path = os.path.join(CSRC, src)
     if not _newer_than(obj, [path] + _headers()):
         return obj, ""
-    cmd = ["nvcc"] + NVCC_FLAGS + (["-Xptxas", "-v"] if verbose else []) + \
+    cmd = [NVCC] + NVCC_FLAGS + (["-Xptxas", "-v"] if verbose else []) + \
           ["-c", path, "-o", obj]
     r = subprocess.run(cmd, capture_output=True, text=True)
     if r.returncode != 0:
@@ -53,23 +69,39 @@ def _compile(src, verbose):
     return obj, r.stderr
 
 
+def _up_to_date(lib, sources):
+    return not _newer_than(lib, [os.path.join(CSRC, f) for f in sources] + _headers())
+
+
+def _library(lib, sources, verbose=False):
+    with concurrent.futures.ThreadPoolExecutor(max_workers=8) as pool:
+        results = list(pool.map(lambda s: _compile(s, verbose), sources))
+    objs = [o for o, _ in results]
+    if verbose:
+        for _, log in results:
+            sys.stderr.write(log)
+    if _newer_than(lib, objs):
+        cmd = [NVCC, "-shared", "-gencode", "arch=compute_100a,code=sm_100a",
+               "-o", lib + ".tmp"] + objs + ["-ldl", "-lpthread",
+                                             "-Xlinker", "--no-undefined"]
+        subprocess.run(cmd, check=True)
+        os.replace(lib + ".tmp", lib)
+    return lib
+
+
 def build(force=False, verbose=False):
     os.makedirs(OBJ, exist_ok=True)
     if force:
         for f in os.listdir(OBJ):
             os.remove(os.path.join(OBJ, f))
-    with concurrent.futures.ThreadPoolExecutor(max_workers=8) as pool:
-        results = list(pool.map(lambda s: _compile(s, verbose), SOURCES))
-    objs = [o for o, _ in results]
-    if verbose:
-        for _, log in results:
-            sys.stderr.write(log)
-    if _newer_than(LIB, objs):
-        cmd = ["nvcc", "-shared", "-gencode", "arch=compute_100a,code=sm_100a",
-               "-o", LIB + ".tmp"] + objs + ["-ldl", "-lpthread"]
-        subprocess.run(cmd, check=True)
-        os.replace(LIB + ".tmp", LIB)
-    return LIB
+    return _library(LIB, SOURCES, verbose)
+
+
+def for_parallel_decoders():
+    if os.path.exists(LIB) and _up_to_date(LIB, SOURCES):
+        return LIB
+    os.makedirs(OBJ, exist_ok=True)
+    return _library(PARALLEL_LIB, PARALLEL_SOURCES)
 
 
 if __name__ == "__main__":

@@ -40,6 +40,10 @@
 
 namespace vxb {
 
+bool tensor_maps_available();
+bool make_map_16(CUtensorMap *map, const void *base, int64_t inner, int64_t rows,
+                 int64_t ld, int box_inner, int box_rows, bool is_bf16);
+
 const char *gemm_16_plain(bool is_bf16, const void *a, int64_t lda,
                           const void *b, int64_t ldb, void *c, int64_t ldc,
                           int64_t m, int64_t n, int64_t k, cudaStream_t stream);
@@ -282,52 +286,6 @@ umma_gemm_kernel(const __grid_constant__ CUtensorMap map_a,
 }
 
 /* ---- host side ------------------------------------------------------------- */
-typedef CUresult (*EncodeTiled)(CUtensorMap *, CUtensorMapDataType, cuuint32_t,
-                                void *, const cuuint64_t *, const cuuint64_t *,
-                                const cuuint32_t *, const cuuint32_t *,
-                                CUtensorMapInterleave, CUtensorMapSwizzle,
-                                CUtensorMapL2promotion, CUtensorMapFloatOOBfill);
-
-EncodeTiled encoder() {
-  static EncodeTiled fn = [] {
-    void *p = nullptr;
-    cudaDriverEntryPointQueryResult q;
-    if (cudaGetDriverEntryPoint("cuTensorMapEncodeTiled", &p, cudaEnableDefault,
-                                &q) != cudaSuccess ||
-        q != cudaDriverEntryPointSuccess) {
-      cudaGetLastError();
-      return (EncodeTiled) nullptr;
-    }
-    return (EncodeTiled)p;
-  }();
-  return fn;
-}
-
-} // namespace
-
-/* A 2-D map over a row-major matrix of 16-bit elements: `inner` contiguous
-   elements per row, `rows` rows `ld` elements apart; boxes of box_inner x
-   box_rows, 128-byte swizzle (box_inner must be 64). */
-bool make_map_16(CUtensorMap *map, const void *base, int64_t inner, int64_t rows,
-                 int64_t ld, int box_inner, int box_rows, bool is_bf16) {
-  EncodeTiled enc = encoder();
-  if (!enc)
-    return false;
-  const cuuint64_t dims[2] = {(cuuint64_t)inner, (cuuint64_t)rows};
-  const cuuint64_t strides[1] = {(cuuint64_t)ld * 2};
-  const cuuint32_t box[2] = {(cuuint32_t)box_inner, (cuuint32_t)box_rows};
-  const cuuint32_t estr[2] = {1, 1};
-  return enc(map,
-             is_bf16 ? CU_TENSOR_MAP_DATA_TYPE_BFLOAT16
-                     : CU_TENSOR_MAP_DATA_TYPE_FLOAT16,
-             2, const_cast<void *>(base), dims, strides, box, estr,
-             CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
-             CU_TENSOR_MAP_L2_PROMOTION_L2_256B,
-             CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
-namespace {
-
 int sm_count() {
   static int n = [] {
     int dev = 0, v = 0;
@@ -413,7 +371,8 @@ const char *gemm_16(bool is_bf16, const void *a, int64_t lda, const void *b,
   /* The tensor-core kernel moves whole 128x256 tiles; below a few tiles, and
      for strides TMA cannot describe, the plain kernel is the one to use. */
   const bool small = m * n < 128 * 256 || k < 64;
-  if (small || !umma_shape_ok(a, lda, b, ldb, c, ldc, m, n, k) || !encoder())
+  if (small || !umma_shape_ok(a, lda, b, ldb, c, ldc, m, n, k) ||
+      !tensor_maps_available())
     return gemm_16_plain(is_bf16, a, lda, b, ldb, c, ldc, m, n, k, stream);
   /* One CTA per 128x256 tile, or a CTA pair per 256x256 tile. The single CTA's
      MMA is held to 77 % of the tensor pipe by its operand fetch and the pair's

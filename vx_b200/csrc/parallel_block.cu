@@ -19,9 +19,11 @@
 namespace vxb {
 namespace {
 
-/* ---- token rows with their position, normalised: a block per row ------------- */
-__global__ void __launch_bounds__(256) position_embed_kernel(const PositionEmbedArgs a) {
-  __shared__ float red[8];
+/* ---- token rows with their position, normalised: a block per row, a thread per
+   pair of values that share an angle ---------------------------------------------- */
+__global__ void __launch_bounds__(1024) position_embed_kernel(const PositionEmbedArgs a) {
+  extern __shared__ __align__(8) float embed_row[]; /* [dim] */
+  __shared__ float red[32];
   chain_release();
   chain_wait();
   const int64_t t = blockIdx.x;
@@ -34,28 +36,39 @@ __global__ void __launch_bounds__(256) position_embed_kernel(const PositionEmbed
     return;
   }
   float ss = 0.0f;
-  for (int i = threadIdx.x; i < a.width; i += blockDim.x) {
-    const int64_t at = (int64_t)token * a.dim + i;
-    const float e = a.table_bf16 ? bf16_val(a.table, at) : ((const float *)a.table)[at];
+#pragma unroll 2
+  for (int k = threadIdx.x; 2 * k < a.width; k += blockDim.x) {
+    /* dim is even, so a pair of the table is one aligned load; the second value
+       of an odd width's last pair is filling */
+    float2 e;
+    if (a.table_bf16) {
+      const uint32_t two =
+          ((const uint32_t *)a.table)[((int64_t)token * a.dim >> 1) + k];
+      e = make_float2(bf_lo(two), bf_hi(two));
+    } else {
+      e = ((const float2 *)a.table)[((int64_t)token * a.dim >> 1) + k];
+    }
     /* the angle in turns: what is left of it after whole turns is exact enough
        in f64 for any position, and small in f32 */
-    const double turns = pos * a.turns[i / 2];
-    const float half_turns = 2.0f * (float)(turns - rint(turns));
-    const float p = i % 2 == 0 ? sinpif(half_turns) : cospif(half_turns);
-    const float v = fmaf(e, a.scale, p);
-    row[i] = v;
-    ss = fmaf(v, v, ss);
+    const double turns = pos * a.turns[k];
+    float sine, cosine;
+    sincospif(2.0f * (float)(turns - rint(turns)), &sine, &cosine);
+    const float v0 = fmaf(e.x, a.scale, sine);
+    const float v1 = 2 * k + 1 < a.width ? fmaf(e.y, a.scale, cosine) : 0.0f;
+    *reinterpret_cast<float2 *>(&embed_row[2 * k]) = make_float2(v0, v1);
+    ss = fmaf(v0, v0, ss);
+    ss = fmaf(v1, v1, ss);
   }
   ss = warp_sum(ss);
   if ((threadIdx.x & 31) == 0)
     red[threadIdx.x >> 5] = ss;
   __syncthreads();
   float total = 0.0f;
-  for (int k = 0; k < 8; ++k) /* fixed order */
+  for (int k = 0; k < (int)blockDim.x / 32; ++k) /* fixed order */
     total += red[k];
   const float inv = 1.0f / sqrtf(total / (float)a.width + a.eps);
-  for (int i = threadIdx.x; i < a.dim; i += blockDim.x) /* its own values again */
-    row[i] = i < a.width ? row[i] * inv * a.gain[i] : 0.0f;
+  for (int i = threadIdx.x; i < a.dim; i += blockDim.x)
+    row[i] = i < a.width ? embed_row[i] * inv * a.gain[i] : 0.0f;
 }
 
 /* ---- after the input GEMM: a thread per (position, eight rows) ---------------- */
@@ -168,7 +181,17 @@ rows_gemm_f32_kernel(const __nv_bfloat16 *terms, const float *w, int t_count, in
 const char *position_embed(const PositionEmbedArgs &a, cudaStream_t stream) {
   if (a.count <= 0)
     return nullptr;
-  launch_chained(position_embed_kernel, dim3(a.count), dim3(256), 0, stream, a);
+  const int smem = a.dim * (int)sizeof(float);
+  if (a.dim % 2 != 0 || ((uintptr_t)a.table & 7))
+    return "a row of the embedding is an even number of values, 8-byte aligned";
+  if (smem > 200 * 1024 ||
+      allow_dynamic_smem((const void *)position_embed_kernel, 200 * 1024) != cudaSuccess)
+    return "a row of the embedding must fit in shared memory (51200 values)";
+  /* few rows: a thread per pair; many: enough blocks are in flight anyway */
+  int threads = a.count > 64 ? 256 : 1024;
+  while (threads > 32 && threads >= a.width)
+    threads /= 2;
+  launch_chained(position_embed_kernel, dim3(a.count), dim3(threads), smem, stream, a);
   return check_launch("the embedding launch");
 }
 

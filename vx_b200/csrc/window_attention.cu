@@ -16,6 +16,7 @@
 #include <cooperative_groups.h>
 
 #include <cstdio>
+#include <cstdlib>
 
 namespace vxb {
 namespace {
@@ -425,10 +426,19 @@ void launch_decode(const WindowAttnArgs &a, dim3 grid, float *out, int64_t out_s
                            out_stride);
   };
   /* few blocks: more warps each, so that a window is a trip or two to memory */
-  if (D4 == 1 && 2 * blocks <= sm_count())
-    go(window_decode_kernel<GH, D4, D4 == 1 ? 16 : 4>, D4 == 1 ? 16 : 4);
-  else if (D4 <= 2 && blocks <= 2 * sm_count())
-    go(window_decode_kernel<GH, D4, D4 <= 2 ? 8 : 4>, D4 <= 2 ? 8 : 4);
+  int warps = 2 * blocks <= sm_count() ? 16 : (blocks <= 2 * sm_count() ? 8 : 4);
+  /* VXB_ATTN_WARPS=4, 8 or 16 pins it (for measurements) */
+  if (const char *pin = getenv("VXB_ATTN_WARPS")) {
+    const int v = atoi(pin);
+    if (v == 4 || v == 8 || v == 16)
+      warps = v;
+  }
+  /* long rows take more shared memory per warp */
+  constexpr int most = 16 / D4;
+  if (warps == 16 && most >= 16)
+    go(window_decode_kernel<GH, D4, most >= 16 ? 16 : 4>, 16);
+  else if (warps >= 8 && most >= 8)
+    go(window_decode_kernel<GH, D4, most >= 8 ? 8 : 4>, 8);
   else
     go(window_decode_kernel<GH, D4, 4>, 4);
 }

@@ -106,6 +106,14 @@ class Llama2cConfig(C.Structure):
                  "vocab_size", "seq_len")]
 
 
+def use(path):
+    """The library to load, before anything has asked for it."""
+    global LIB_PATH
+    if _lib is not None and path != LIB_PATH:
+        raise RuntimeError("%s is loaded already" % LIB_PATH)
+    LIB_PATH = path
+
+
 def lib():
     global _lib
     if _lib is not None:
