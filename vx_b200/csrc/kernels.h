@@ -358,11 +358,12 @@ const char *rows_gemm(const void *terms, const void *w, int t, int n, int cols,
                       float *partials, int *splits_out, cudaStream_t stream);
 /* The same GEMM for any two bf16 matrices: terms [t, term_cols], w [n, w_cols];
    K block kb of the terms meets K block kb mod (w_cols / 64) of w (term_cols
-   need not be a multiple of w_cols). */
+   need not be a multiple of w_cols). splits: how many runs, 0 for what takes
+   least time (rows_gemm_splits_of). */
 int rows_gemm_splits_of(int t, int n, int64_t term_cols);
 const char *rows_gemm_of(const void *terms, int64_t term_cols, const void *w,
                          int64_t w_cols, int t, int n, float *partials,
-                         int *splits_out, cudaStream_t stream);
+                         int *splits_out, cudaStream_t stream, int splits = 0);
 /* For quantised weights on that GEMM. Q4_0: a matrix [n, cols] as [n, 2 cols]
    bf16 = w1 | w2 with w1 + w2 = (code - 8) * scale exactly, against terms spread
    to x1 | x1 | x2 | x2 | x3 | x3 (segments 6, from {0,0,1,1,2,2}). fp8: the f32

@@ -750,7 +750,7 @@ const char *rows_gemm(const void *terms, const void *w, int t, int n, int cols,
 
 const char *rows_gemm_of(const void *terms, int64_t term_cols, const void *w,
                          int64_t w_cols, int t, int n, float *partials,
-                         int *splits_out, cudaStream_t stream) {
+                         int *splits_out, cudaStream_t stream, int splits) {
   if (term_cols % BK != 0 || w_cols % BK != 0)
     return "the multi-position projections need columns in multiples of 64";
   if (allow_dynamic_smem((const void *)rows_gemm_kernel, SMEM_BYTES) != cudaSuccess)
@@ -765,7 +765,7 @@ const char *rows_gemm_of(const void *terms, int64_t term_cols, const void *w,
   g.n = n;
   g.k_blocks = (int)(term_cols / BK);
   g.w_blocks = (int)(w_cols / BK);
-  g.splits = rows_gemm_splits_of(t, n, term_cols);
+  g.splits = splits > 0 ? splits : rows_gemm_splits_of(t, n, term_cols);
   g.partials = partials;
   *splits_out = g.splits;
   int pairs = resident_pairs();
