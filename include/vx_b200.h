@@ -369,7 +369,79 @@ typedef struct {
 
 /* NULL with vx_b200_last_error() for sizes it cannot take. */
 vx_decoder *vx_decoder_create_parallel(const vx_parallel_config *config);
-/* The next `count` tokens of a one-sequence decoder of parallel blocks, and the
+
+/* ---- decoders of layers around several residual streams -------------------------
+ * The residual is `streams` rows x_s, all equal to scale * embedding row at the
+ * start. A layer is a mixer and then a feed-forward (or none), each of which reads the
+ * RMSNorm of sum_s in[s] x_s and puts its output y back: x_t <- sum_s mix[s][t] x_s +
+ * out[t] y, from the old x_s (one stream and ones: the ordinary residual). Mixers:
+ *   VX_MIXER_LATENT  attention over a sliding window, queries through a latent of
+ *     q_rank values, keys and values out of a latent of kv_rank values, one rotated
+ *     key part for all heads; cached are the normalised latent and that part.
+ *   VX_MIXER_GATED_LINEAR  per head a state [dim][vdim], S <- diag(alpha) S + k v^T,
+ *     o = S^T q, alpha = sigmoid(W_a2 W_a1 h + bias)^(1 / tau) per key channel; o
+ *     through an RMSNorm per head, times silu(W_g h).
+ * The feed-forward is W_down gelu(W_up h), the exact gelu. The logits are
+ * cap * tanh(scale * head norm(sum_s x_s) / cap). Layers may differ in kind and size;
+ * a layer that runs several times is listed as often, with the same pointers. No
+ * counterpart in the reference. Everything that takes a decoder of parallel blocks
+ * takes these: the V cache is NULL, and the K cache holds the listed layers' rings
+ * ([sequence][rows][kv_rank + rot_dim], rows = min(max_seq, window - 1 +
+ * prefill_rows), position t in row t mod rows) and states
+ * ([sequence][heads][dim][vdim]) one after another.
+ *
+ * Device pointers; the caller owns the memory. Matrices are bf16 or f32, everything
+ * else f32 (turns f64). dim, rot_dim, vdim, a_rank: filled up to multiples of 8;
+ * heads * vdim, q_rank, kv_rank, hidden: of 64; with zeros in the rows, columns and
+ * gains that fill up. */
+enum { VX_MIXER_LATENT = 1, VX_MIXER_GATED_LINEAR = 2 };
+typedef struct {
+  const float *in;  /* [streams] */
+  const float *mix; /* [streams from][streams to] */
+  const float *out; /* [streams] */
+} vx_stream_mix;
+typedef struct {
+  int32_t kind; /* VX_MIXER_* */
+  int32_t heads, dim, vdim;
+  /* latent: dim is the unrotated part; q_mean, kv_mean: how many values of the
+     latents are the model's, which is what their norms' means are over */
+  int32_t rot_dim, q_rank, q_mean, kv_rank, kv_mean, window;
+  /* gated linear: v_mean as above */
+  int32_t a_rank, v_mean;
+  int32_t hidden;     /* of the feed-forward; 0: none */
+  float scale;        /* of the scores; of q */
+  float inv_tau;      /* gated linear */
+  const float *norm1; /* [dim of the model] */
+  /* latent: rows q_rank | kv_rank | rot_dim; gated linear: q | k | v | gate | a1 */
+  const void *w_in;
+  const void *w_o; /* [dim of the model, heads * vdim] */
+  const float *q_norm, *kv_norm; /* latent: [q_rank], [kv_rank] */
+  const void *w_uq;   /* [heads * (dim + rot_dim), q_rank], a head's rotated rows last */
+  const void *w_ukv;  /* [heads * (dim + vdim), kv_rank], a head's key rows first */
+  const void *w_uk_t; /* [heads * kv_rank, dim]: each head's key rows transposed */
+  const double *turns; /* [rot_dim / 2]: how much of a full turn the pair (2i, 2i + 1)
+                          advances per position */
+  const float *a2, *a2_bias; /* gated linear: [heads * dim, a_rank], [heads * dim] */
+  const float *o_norm;       /* gated linear: [vdim] */
+  const float *norm2;
+  const void *w_up, *w_down; /* [hidden, .], [., hidden] */
+  vx_stream_mix hc1, hc2;    /* of the mixer and of the feed-forward */
+} vx_stream_layer;
+typedef struct {
+  /* as in vx_parallel_config */
+  int32_t width, dim, n_layers, vocab, vocab_rows, max_seq, weights_bf16, batch,
+      prefill_rows;
+  int32_t streams; /* 1 to 32 */
+  float eps, embed_scale, logit_scale;
+  float logit_cap; /* 0: none */
+  const void *embed, *classifier;
+  const float *final_norm;
+  const vx_stream_layer *layers; /* host memory, n_layers of them */
+} vx_stream_config;
+/* NULL with vx_b200_last_error() for sizes it cannot take. */
+vx_decoder *vx_decoder_create_streams(const vx_stream_config *config);
+
+/* The next `count` tokens of a one-sequence decoder of one of these two kinds, and the
    logits after n_want of them: want[i] (host, ascending) counts from the first of
    these tokens, and row i of logits (host, [n_want, vocab] f32) belongs to it.
    Waits for the GPU when n_want > 0. Returns count, or -1 with

@@ -1,8 +1,9 @@
 """Build vx_b200/libvx_cuda_dispatch.so from csrc/*.cu with nvcc for sm_100a.
 
-for_parallel_decoders() gives a library that can serve decoders of parallel blocks:
-the whole one where it is built and up to date, else a smaller one of the same
-objects, libvx_parallel_decoder.so, which takes less compiling.
+for_parallel_decoders() and for_stream_decoders() give a library that can serve one
+kind of decoder (of parallel blocks; of several residual streams): the whole one where
+it is built and up to date, else a smaller one of the same objects,
+libvx_parallel_decoder.so or libvx_stream_decoder.so, which takes less compiling.
 
 The library is built in-tree, so that it travels with the source directory; it
 links the CUDA runtime statically and opens libcuda.so.1 and libnccl.so.2 at
@@ -20,6 +21,7 @@ CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(HERE, "_obj")
 LIB = os.path.join(HERE, "libvx_cuda_dispatch.so")
 PARALLEL_LIB = os.path.join(HERE, "libvx_parallel_decoder.so")
+STREAM_LIB = os.path.join(HERE, "libvx_stream_decoder.so")
 NVCC = shutil.which("nvcc") or "/usr/local/cuda/bin/nvcc"
 
 SOURCES = ["rowdot_quant.cu", "rowdot_bf16.cu", "rowdot_f32.cu", "nn_kernels.cu",
@@ -28,13 +30,19 @@ SOURCES = ["rowdot_quant.cu", "rowdot_bf16.cu", "rowdot_f32.cu", "nn_kernels.cu"
            "flash_attn_v2.cu", "static_scratch.cu", "rowdot_umma.cu", "prefill.cu",
            "quantize.cu", "step_kernel.cu", "gemm_f32_split.cu", "moe_group.cu",
            "moe_grouped.cu", "gemm_fp8_rows.cu", "window_attention.cu",
-           "parallel_block.cu", "tensor_map.cu"]
-# what a decoder of parallel blocks runs and loads its weights with; absent.cu
-# stands for the rest
-PARALLEL_SOURCES = ["rowdot_bf16.cu", "rowdot_f32.cu", "nn_kernels.cu", "dispatch.cu",
-                    "nn_api.cu", "decoder.cu", "decoder_parallel.cu", "prefill.cu",
-                    "window_attention.cu", "parallel_block.cu", "tensor_map.cu",
-                    "absent.cu"]
+           "parallel_block.cu", "tensor_map.cu", "decoder_streams.cu",
+           "latent_attention.cu", "gated_linear.cu", "residual_streams.cu",
+           "rowdot_streams_bf16.cu", "rowdot_streams_f32.cu"]
+# what the decoders run and load their weights with; absent*.cu stand for the rest
+_DECODER_SOURCES = ["nn_kernels.cu", "dispatch.cu", "nn_api.cu", "decoder.cu",
+                    "prefill.cu", "parallel_block.cu", "tensor_map.cu", "absent.cu"]
+PARALLEL_SOURCES = _DECODER_SOURCES + [
+    "rowdot_bf16.cu", "rowdot_f32.cu", "decoder_parallel.cu", "window_attention.cu",
+    "absent_streams.cu"]
+STREAM_SOURCES = _DECODER_SOURCES + [
+    "rowdot_streams_bf16.cu", "rowdot_streams_f32.cu", "decoder_streams.cu",
+    "latent_attention.cu", "gated_linear.cu", "residual_streams.cu",
+    "absent_parallel.cu"]
 NVCC_FLAGS = ["-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3",
               "-std=c++17", "-Xcompiler", "-fPIC", "-Xcompiler", "-Wall",
               "-I" + os.path.join(ROOT, "include"),
@@ -97,11 +105,19 @@ def build(force=False, verbose=False):
     return _library(LIB, SOURCES, verbose)
 
 
-def for_parallel_decoders():
+def _whole_or(lib, sources):
     if os.path.exists(LIB) and _up_to_date(LIB, SOURCES):
         return LIB
     os.makedirs(OBJ, exist_ok=True)
-    return _library(PARALLEL_LIB, PARALLEL_SOURCES)
+    return _library(lib, sources)
+
+
+def for_parallel_decoders():
+    return _whole_or(PARALLEL_LIB, PARALLEL_SOURCES)
+
+
+def for_stream_decoders():
+    return _whole_or(STREAM_LIB, STREAM_SOURCES)
 
 
 if __name__ == "__main__":

@@ -1,21 +1,10 @@
-/* absent.cu -- the launchers that a library for decoders of parallel blocks leaves
- * out (vx_b200/build.py): each refuses, and the status words are 0.  The whole
- * library has the kernels themselves in their place. */
-#include "kernels.h"
-#include "nn_device.cuh"
-#include "vx_b200.h"
+/* absent.cu -- the launchers that the libraries for one kind of decoder leave out
+ * (vx_b200/build.py): each refuses, and the status words are 0.  The whole library has
+ * the kernels themselves in their place.  absent_parallel.cu and absent_streams.cu
+ * stand for the other kind of decoder. */
+#include "absent.h"
 
 namespace vxb {
-
-void set_last_error(const char *why);
-
-#define NOT_HERE(name)                                                                   \
-  name " is not part of this library, which serves decoders of parallel blocks; build "  \
-       "the whole one (python -m vx_b200.build)"
-#define ABSENT(name, ...)                                                                \
-  const char *name(__VA_ARGS__) { return NOT_HERE(#name); }
-
-using Stream = cudaStream_t;
 
 ABSENT(gemm_f32, const float *, int64_t, const float *, int64_t, float *, int64_t, int64_t,
        int64_t, int64_t, Stream)

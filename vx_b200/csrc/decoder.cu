@@ -409,6 +409,10 @@ void record_step(vx_decoder *d, int max_pos) {
     decoder_record_parallel_step(d);
     return;
   }
+  if (d->streams) {
+    decoder_record_stream_step(d);
+    return;
+  }
   if (d->one_kernel) {
     record_one_kernel_step(d);
     return;
@@ -781,6 +785,7 @@ vx_decoder *vx_decoder_create(const vx_decoder_config *config,
   }
   d->logit_stride = d->vocab_local;
   d->par = nullptr;
+  d->streams = nullptr;
   d->one_kernel = false;
   d->step_ops = nullptr;
   d->n_step_ops = 0;
@@ -834,6 +839,7 @@ void vx_decoder_destroy(vx_decoder *d) {
                   (void *)d->step_trace})
     cudaFree(p);
   decoder_free_parallel(d);
+  decoder_free_streams(d);
   cudaFree(d->owned_weights);
   cudaStreamDestroy(d->stream);
   delete d;
@@ -863,7 +869,7 @@ int32_t vx_decoder_step(vx_decoder *d, const int32_t *tokens_in,
   const int pos = d->host_pos;
   if (pos >= d->c.max_seq)
     stop("vx_decoder_step: position %d is past max_seq %d", pos, d->c.max_seq);
-  cudaGraphExec_t exec = graph_for(d, d->one_kernel || d->par ? 0 : pos / 256);
+  cudaGraphExec_t exec = graph_for(d, d->one_kernel || d->par || d->streams ? 0 : pos / 256);
   if (tokens_in)
     CUDA_OK(cudaMemcpyAsync(d->tokens, tokens_in, d->c.batch * sizeof(int32_t),
                             cudaMemcpyHostToDevice, d->stream));
@@ -879,6 +885,42 @@ int32_t vx_decoder_step(vx_decoder *d, const int32_t *tokens_in,
   return pos;
 }
 
+int32_t vx_decoder_prefill_logits(vx_decoder *d, const int32_t *tokens, int32_t count,
+                                  const int32_t *want, int32_t n_want, float *logits) {
+  const RowsPlan *rows = d->par ? &d->par->rows : d->streams ? &d->streams->rows : nullptr;
+  if (!rows || d->c.batch != 1) {
+    vxb::set_last_error("vx_decoder_prefill_logits: needs a decoder of parallel blocks "
+                        "or of several streams, with one sequence");
+    return -1;
+  }
+  if (count < 0 || (count && !tokens) || d->host_pos + count > d->c.max_seq) {
+    vxb::set_last_error("vx_decoder_prefill_logits: the tokens do not fit max_seq");
+    return -1;
+  }
+  bool ascending = n_want >= 0 && (n_want == 0 || (want && logits));
+  for (int i = 0; ascending && i < n_want; ++i)
+    ascending = want[i] < count && want[i] > (i ? want[i - 1] : -1);
+  if (!ascending) {
+    vxb::set_last_error("vx_decoder_prefill_logits: want must be ascending places among "
+                        "the tokens");
+    return -1;
+  }
+  std::vector<int32_t> here;
+  int done = 0;
+  for (int at = 0; at < count;) {
+    const int t = std::min(count - at, rows->prefill_rows);
+    here.clear();
+    while (done + (int)here.size() < n_want && want[done + here.size()] < at + t)
+      here.push_back(want[done + here.size()] - at);
+    (d->par ? decoder_parallel_rows : decoder_stream_rows)(
+        d, tokens + at, t, here.data(), (int)here.size(),
+        logits ? logits + (int64_t)done * d->c.vocab : nullptr);
+    done += (int)here.size();
+    at += t;
+  }
+  return count;
+}
+
 /* A run of prompt tokens of a one-sequence decoder, all positions at once: the
    positions are the rows of tensor-core GEMMs (prefill.cu; the reference's form
    of this are the multi-row kernels of nn.vx:2317-3066), every position writes
@@ -888,7 +930,7 @@ int32_t vx_decoder_step(vx_decoder *d, const int32_t *tokens_in,
    there are fewer than 32: single steps are as fast then), or -1 with
    vx_b200_last_error() when this decoder cannot do it. */
 int32_t vx_decoder_prefill(vx_decoder *d, const int32_t *tokens, int32_t count) {
-  if (d->par)
+  if (d->par || d->streams)
     return vx_decoder_prefill_logits(d, tokens, count, nullptr, 0, nullptr);
   const vx_decoder_config &c = d->c;
   const int hd = c.head_dim;
@@ -1282,14 +1324,15 @@ float *vx_decoder_kv_cache(vx_decoder *d, int32_t which) {
 int32_t vx_decoder_logits_pitch(const vx_decoder *d) { return d->logit_stride; }
 
 int64_t vx_decoder_kv_cache_bytes(const vx_decoder *d) {
-  if (d->par)
-    return d->par->cache_floats * (int64_t)sizeof(float);
+  if (d->par || d->streams)
+    return (d->par ? d->par->cache_floats : d->streams->cache_floats) *
+           (int64_t)sizeof(float);
   return d->cache_layer_stride * d->c.n_layers * (int64_t)sizeof(float);
 }
 
 int32_t vx_decoder_adopt_kv(vx_decoder *d, const float *k, const float *v,
                             int32_t positions) {
-  if (!k || (!v && !d->par) || positions < 0 || positions > d->c.max_seq) {
+  if (!k || (!v && !d->par && !d->streams) || positions < 0 || positions > d->c.max_seq) {
     vxb::set_last_error("vx_decoder_adopt_kv: needs both caches and 0 <= "
                         "positions <= max_seq");
     return -1;
@@ -1307,9 +1350,21 @@ int32_t vx_decoder_adopt_kv(vx_decoder *d, const float *k, const float *v,
             cudaMemcpyDefault, d->stream));
       }
     }
-  const size_t run = d->par ? 0
-                            : (size_t)positions * d->kv_local * d->c.head_dim *
-                                  sizeof(float);
+  if (d->streams) /* rings likewise; a state is what the last position left */
+    for (const StreamLayer &layer : d->streams->layers) {
+      const int rows = positions < layer.cache_rows ? positions : layer.cache_rows;
+      const size_t row = layer.l.kind == VX_MIXER_LATENT
+                             ? (size_t)(layer.l.kv_rank + layer.l.rot_dim)
+                             : (size_t)layer.batch_stride;
+      for (int b = 0; b < d->c.batch && rows; ++b) {
+        const int64_t at = layer.at + b * layer.batch_stride;
+        CUDA_OK(cudaMemcpyAsync(d->k_cache + at, k + at, rows * row * sizeof(float),
+                                cudaMemcpyDefault, d->stream));
+      }
+    }
+  const size_t run = d->par || d->streams ? 0
+                                          : (size_t)positions * d->kv_local *
+                                                d->c.head_dim * sizeof(float);
   for (int l = 0; l < d->c.n_layers && run; ++l)
     for (int b = 0; b < d->c.batch; ++b) {
       const int64_t at = l * d->cache_layer_stride + b * d->cache_batch_stride;

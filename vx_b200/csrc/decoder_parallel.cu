@@ -13,6 +13,7 @@
  * The cache is a ring per layer and sequence: a window never needs more than its
  * own size and the portion being read, whatever the length of the sequence.
  */
+#include "decoder_rows.h"
 #include "decoder_state.h"
 #include "kernels.h"
 #include "vx_b200.h"
@@ -79,28 +80,6 @@ const float *normed(vx_decoder *d, const float *gain, int &launches) {
   return d->xn;
 }
 
-template <typename T> void grow(T *&p, size_t count) {
-  cudaFree(p);
-  p = dev_alloc<T>(count);
-}
-void grow_terms(void *&p, size_t values) {
-  cudaFree(p);
-  p = dev_alloc<uint16_t>(values * 3);
-}
-
-/* One product of t positions: partials[run][t][n]. */
-void rows_product(vx_decoder *d, const void *terms, const void *w, int t, int n, int cols,
-                  int *runs, const char *what) {
-  *runs = 1;
-  need(d->c.weights_bf16
-           ? vxb::rows_gemm(terms, w, t, n, cols, d->rows_partials, runs, d->stream)
-           : vxb::rows_gemm_f32(terms, (const float *)w, t, n, cols, d->rows_partials,
-                                d->stream),
-       what);
-}
-
-constexpr int WANT_GROUP = 256; /* positions whose logits are computed together */
-
 /* Room for t positions and for the logits of n_want of them. */
 void make_room(vx_decoder *d, int t, int n_want) {
   ParallelPlan &p = *d->par;
@@ -114,125 +93,14 @@ void make_room(vx_decoder *d, int t, int n_want) {
     grow(d->rows_tokens, t);
     d->rows_cap = t;
   }
-  const int group = std::min(n_want, WANT_GROUP);
-  if (group > p.want_cap) {
-    grow(p.want, group);
-    grow_terms(p.want_terms, (size_t)group * c.dim);
-    grow(p.want_logits, (size_t)group * p.vocab_rows);
-    p.want_cap = group;
-  }
-  /* The runs of a product depend on how many positions it has, so the sums of
-     few positions can take more room than those of many. */
-  size_t most = 0;
-  auto sums = [&](int positions, int n, int cols) {
-    const size_t runs = c.weights_bf16 ? vxb::rows_gemm_splits(positions, n, cols) : 1;
-    most = std::max(most, runs * positions * n);
-  };
+  SumsRoom sums{d, 0};
   for (const ParallelLayer &l : p.layers) {
-    sums(t, l.in_rows, c.dim);
-    sums(t, l.gate_row - l.k_row, c.dim);
-    sums(t, c.dim, l.out_cols);
+    sums.add(t, l.in_rows, c.dim);
+    sums.add(t, l.gate_row - l.k_row, c.dim);
+    sums.add(t, c.dim, l.out_cols);
   }
-  if (n_want > 0) {
-    sums(group, p.vocab_rows, c.dim);
-    if (n_want % WANT_GROUP)
-      sums(n_want % WANT_GROUP, p.vocab_rows, c.dim);
-  }
-  if (most > d->rows_partial_floats) {
-    grow(d->rows_partials, most);
-    d->rows_partial_floats = most;
-  }
-}
-
-/* The next t positions of the sequence through all layers. */
-void rows_pass(vx_decoder *d, const int32_t *tokens, int t, const int32_t *want,
-               int n_want, float *logits) {
-  ParallelPlan &p = *d->par;
-  const vx_decoder_config &c = d->c;
-  cudaStream_t s = d->stream;
-  const int w_bytes = c.weights_bf16 ? 2 : 4;
-  make_room(d, t, n_want);
-  CUDA_OK(cudaMemcpyAsync(d->rows_tokens, tokens, (size_t)t * sizeof(int32_t),
-                          cudaMemcpyHostToDevice, s));
-  need(vxb::position_embed(embed_args(d, d->rows_x, d->rows_tokens, t, false), s),
-       "embed");
-  const bool fuse_norm = c.dim <= 8192;
-  need(vxb::rows_norm_terms(d->rows_terms, d->rows_x, NormGain(p.layers[0].norm, p.width),
-                            t, c.dim, c.eps, s),
-       "RMSNorm");
-  int runs = 1;
-  for (int i = 0; i < c.n_layers; ++i) {
-    /* rows_terms hold the terms of this layer's h */
-    const ParallelLayer &l = p.layers[i];
-    const bool last = i == c.n_layers - 1;
-    vxb::FanOut fan{};
-    fan.k_row = l.k_row;
-    fan.gate_row = l.gate_row;
-    fan.up_row = l.up_row;
-    fan.cache_rows = l.cache_rows;
-    fan.gate = p.rows_gate;
-    fan.gate_stride = p.q_max;
-    float *ring = d->k_cache + l.cache_at;
-    const int att_cols = l.q_heads * l.head_dim;
-    if (last && n_want == 0) {
-      /* nothing but the keys of the last layer is read by anyone later */
-      const int k_rows = l.gate_row - l.k_row;
-      fan.k_row = 0;
-      fan.gate_row = fan.up_row = k_rows;
-      rows_product(d, d->rows_terms,
-                   (const char *)l.w_in + (int64_t)l.k_row * c.dim * w_bytes, t, k_rows,
-                   c.dim, &runs, "the keys");
-      need(vxb::rows_fan_finish(d->rows_partials, runs, t, k_rows, fan, d->positions,
-                                d->rows_q, p.q_max, ring, p.rows_mixed_terms, l.out_cols,
-                                att_cols, s),
-           "the ring's new rows");
-      break;
-    }
-    rows_product(d, d->rows_terms, l.w_in, t, l.in_rows, c.dim, &runs,
-                 "the input projection");
-    need(vxb::rows_fan_finish(d->rows_partials, runs, t, l.in_rows, fan, d->positions,
-                              d->rows_q, p.q_max, ring, p.rows_mixed_terms, l.out_cols,
-                              att_cols, s),
-         "the parts of the input projection");
-    need(vxb::window_attention_rows(attention_args(d, l, d->rows_q, p.rows_gate), t,
-                                    p.rows_mixed_terms, l.out_cols, s),
-         "attention");
-    rows_product(d, p.rows_mixed_terms, l.w_out, t, c.dim, l.out_cols, &runs,
-                 "the output projection");
-    if (!last && fuse_norm) {
-      need(vxb::rows_residual_norm(d->rows_terms, d->rows_x, d->rows_partials, runs, t,
-                                   NormGain(p.layers[i + 1].norm, p.width), c.dim, c.eps,
-                                   s),
-           "the residual add and RMSNorm");
-      continue;
-    }
-    need(vxb::rows_residual_finish(d->rows_x, d->rows_partials, runs, t, c.dim, s),
-         "the residual add");
-    if (!last)
-      need(vxb::rows_norm_terms(d->rows_terms, d->rows_x,
-                                NormGain(p.layers[i + 1].norm, p.width), t, c.dim, c.eps,
-                                s),
-           "RMSNorm");
-  }
-  for (int at = 0; at < n_want; at += WANT_GROUP) {
-    const int n = std::min(WANT_GROUP, n_want - at);
-    CUDA_OK(cudaMemcpyAsync(p.want, want + at, n * sizeof(int32_t),
-                            cudaMemcpyHostToDevice, s));
-    need(vxb::rows_norm_terms(p.want_terms, d->rows_x, NormGain(p.final_norm, p.width), n,
-                              c.dim, c.eps, s, p.want),
-         "RMSNorm");
-    rows_product(d, p.want_terms, d->lm_head, n, p.vocab_rows, c.dim, &runs,
-                 "the logits");
-    need(vxb::rows_sum(p.want_logits, d->rows_partials, runs, n, p.vocab_rows, s),
-         "the logits");
-    CUDA_OK(cudaMemcpy2DAsync(logits + (int64_t)at * c.vocab, c.vocab * sizeof(float),
-                              p.want_logits, p.vocab_rows * sizeof(float),
-                              c.vocab * sizeof(float), n, cudaMemcpyDeviceToHost, s));
-    const cudaError_t e = cudaStreamSynchronize(s);
-    if (e != cudaSuccess)
-      stop("a kernel of the decoder faulted: %s", cudaGetErrorString(e));
-  }
-  decoder_advance(d, t);
+  sums.add_logits(n_want, p.vocab_rows, c.dim);
+  make_rows_room(d, p.rows, sums, n_want, p.vocab_rows);
 }
 
 /* A sentence saying why not, or NULL. */
@@ -336,14 +204,91 @@ void decoder_record_parallel_step(vx_decoder *d) {
   decoder_record_tail(d, launches + 1);
 }
 
+void decoder_parallel_rows(vx_decoder *d, const int32_t *tokens, int t,
+                           const int32_t *want, int n_want, float *logits) {
+  ParallelPlan &p = *d->par;
+  const vx_decoder_config &c = d->c;
+  cudaStream_t s = d->stream;
+  const int w_bytes = c.weights_bf16 ? 2 : 4;
+  make_room(d, t, n_want);
+  CUDA_OK(cudaMemcpyAsync(d->rows_tokens, tokens, (size_t)t * sizeof(int32_t),
+                          cudaMemcpyHostToDevice, s));
+  need(vxb::position_embed(embed_args(d, d->rows_x, d->rows_tokens, t, false), s),
+       "embed");
+  const bool fuse_norm = c.dim <= 8192;
+  need(vxb::rows_norm_terms(d->rows_terms, d->rows_x, NormGain(p.layers[0].norm, p.width),
+                            t, c.dim, c.eps, s),
+       "RMSNorm");
+  int runs = 1;
+  for (int i = 0; i < c.n_layers; ++i) {
+    /* rows_terms hold the terms of this layer's h */
+    const ParallelLayer &l = p.layers[i];
+    const bool last = i == c.n_layers - 1;
+    vxb::FanOut fan{};
+    fan.k_row = l.k_row;
+    fan.gate_row = l.gate_row;
+    fan.up_row = l.up_row;
+    fan.cache_rows = l.cache_rows;
+    fan.gate = p.rows_gate;
+    fan.gate_stride = p.q_max;
+    float *ring = d->k_cache + l.cache_at;
+    const int att_cols = l.q_heads * l.head_dim;
+    if (last && n_want == 0) {
+      /* nothing but the keys of the last layer is read by anyone later */
+      const int k_rows = l.gate_row - l.k_row;
+      fan.k_row = 0;
+      fan.gate_row = fan.up_row = k_rows;
+      rows_product(d, d->rows_terms,
+                   (const char *)l.w_in + (int64_t)l.k_row * c.dim * w_bytes, t, k_rows,
+                   c.dim, &runs, "the keys");
+      need(vxb::rows_fan_finish(d->rows_partials, runs, t, k_rows, fan, d->positions,
+                                d->rows_q, p.q_max, ring, p.rows_mixed_terms, l.out_cols,
+                                att_cols, s),
+           "the ring's new rows");
+      break;
+    }
+    rows_product(d, d->rows_terms, l.w_in, t, l.in_rows, c.dim, &runs,
+                 "the input projection");
+    need(vxb::rows_fan_finish(d->rows_partials, runs, t, l.in_rows, fan, d->positions,
+                              d->rows_q, p.q_max, ring, p.rows_mixed_terms, l.out_cols,
+                              att_cols, s),
+         "the parts of the input projection");
+    need(vxb::window_attention_rows(attention_args(d, l, d->rows_q, p.rows_gate), t,
+                                    p.rows_mixed_terms, l.out_cols, s),
+         "attention");
+    rows_product(d, p.rows_mixed_terms, l.w_out, t, c.dim, l.out_cols, &runs,
+                 "the output projection");
+    if (!last && fuse_norm) {
+      need(vxb::rows_residual_norm(d->rows_terms, d->rows_x, d->rows_partials, runs, t,
+                                   NormGain(p.layers[i + 1].norm, p.width), c.dim, c.eps,
+                                   s),
+           "the residual add and RMSNorm");
+      continue;
+    }
+    need(vxb::rows_residual_finish(d->rows_x, d->rows_partials, runs, t, c.dim, s),
+         "the residual add");
+    if (!last)
+      need(vxb::rows_norm_terms(d->rows_terms, d->rows_x,
+                                NormGain(p.layers[i + 1].norm, p.width), t, c.dim, c.eps,
+                                s),
+           "RMSNorm");
+  }
+  rows_logits(d, p.rows, want, n_want, logits, p.vocab_rows, 1.0f, 0.0f, [&](int n) {
+    return vxb::rows_norm_terms(p.rows.want_terms, d->rows_x,
+                                NormGain(p.final_norm, p.width), n, c.dim, c.eps, s,
+                                p.rows.want);
+  });
+  decoder_advance(d, t);
+}
+
 void decoder_free_parallel(vx_decoder *d) {
   if (!d->par)
     return;
   ParallelPlan &p = *d->par;
   for (void *m : {(void *)p.gate, (void *)p.mixed, (void *)p.rows_gate,
-                  p.rows_mixed_terms, (void *)p.want, p.want_terms,
-                  (void *)p.want_logits})
+                  p.rows_mixed_terms})
     cudaFree(m);
+  free_rows(p.rows);
   delete d->par;
 }
 
@@ -374,7 +319,7 @@ vx_decoder *vx_decoder_create_parallel(const vx_parallel_config *config) {
   d->lm_head = pc.classifier;
   p->width = pc.width;
   p->vocab_rows = pc.vocab_rows;
-  p->prefill_rows = std::min(pc.prefill_rows ? pc.prefill_rows : 2048, pc.max_seq);
+  p->rows.prefill_rows = std::min(pc.prefill_rows ? pc.prefill_rows : 2048, pc.max_seq);
   p->embed_scale = pc.embed_scale;
   p->embed_norm = pc.embed_norm;
   p->final_norm = pc.final_norm;
@@ -386,7 +331,7 @@ vx_decoder *vx_decoder_create_parallel(const vx_parallel_config *config) {
     l.kv_heads = from.kv_heads;
     l.head_dim = from.head_dim;
     l.window = std::min(from.window, pc.max_seq);
-    l.cache_rows = std::min(pc.max_seq, l.window - 1 + p->prefill_rows);
+    l.cache_rows = std::min(pc.max_seq, l.window - 1 + p->rows.prefill_rows);
     l.scale = from.score_scale;
     const int att = l.q_heads * l.head_dim;
     l.k_row = att;
@@ -419,40 +364,6 @@ vx_decoder *vx_decoder_create_parallel(const vx_parallel_config *config) {
   CUDA_OK(cudaStreamCreateWithFlags(&d->stream, cudaStreamNonBlocking));
   CUDA_OK(cudaDeviceSynchronize());
   return d;
-}
-
-int32_t vx_decoder_prefill_logits(vx_decoder *d, const int32_t *tokens, int32_t count,
-                                  const int32_t *want, int32_t n_want, float *logits) {
-  if (!d->par || d->c.batch != 1) {
-    vxb::set_last_error("vx_decoder_prefill_logits: needs a decoder of parallel blocks "
-                        "with one sequence");
-    return -1;
-  }
-  if (count < 0 || (count && !tokens) || d->host_pos + count > d->c.max_seq) {
-    vxb::set_last_error("vx_decoder_prefill_logits: the tokens do not fit max_seq");
-    return -1;
-  }
-  bool ascending = n_want >= 0 && (n_want == 0 || (want && logits));
-  for (int i = 0; ascending && i < n_want; ++i)
-    ascending = want[i] < count && want[i] > (i ? want[i - 1] : -1);
-  if (!ascending) {
-    vxb::set_last_error("vx_decoder_prefill_logits: want must be ascending places among "
-                        "the tokens");
-    return -1;
-  }
-  std::vector<int32_t> here;
-  int done = 0;
-  for (int at = 0; at < count;) {
-    const int t = std::min(count - at, d->par->prefill_rows);
-    here.clear();
-    while (done + (int)here.size() < n_want && want[done + here.size()] < at + t)
-      here.push_back(want[done + here.size()] - at);
-    rows_pass(d, tokens + at, t, here.data(), (int)here.size(),
-              logits ? logits + (int64_t)done * d->c.vocab : nullptr);
-    done += (int)here.size();
-    at += t;
-  }
-  return count;
 }
 
 } /* extern "C" */

@@ -1,6 +1,7 @@
 /* decoder_state.h -- what the source files of the decoder share: its state and
  * how it stops.  decoder.cu holds the Llama-2 decoders and the entry points,
- * decoder_parallel.cu the decoders of parallel blocks. */
+ * decoder_parallel.cu the decoders of parallel blocks, decoder_streams.cu those of
+ * layers around a residual of several streams. */
 #ifndef VXB_DECODER_STATE_H
 #define VXB_DECODER_STATE_H
 
@@ -16,6 +17,8 @@
 namespace vxb {
 void set_last_error(const char *why);
 } // namespace vxb
+
+struct vx_decoder;
 
 namespace {
 
@@ -58,6 +61,17 @@ struct PickPeers {
   PickSlot *slots[vxb::kMaxTpRanks];
 };
 
+/* What decoders that give logits of any position keep for the positions of a prompt
+   (decoder_rows.h). */
+struct RowsPlan {
+  int prefill_rows; /* positions that go through the layers together at most */
+  /* of the positions whose logits are asked for: want_cap of them */
+  int32_t *want;
+  void *want_terms;
+  float *want_logits;
+  int want_cap;
+};
+
 /* One parallel block: where its matrices are cut and where its keys are. */
 struct ParallelLayer {
   int q_heads, kv_heads, head_dim;
@@ -72,7 +86,8 @@ struct ParallelLayer {
 };
 struct ParallelPlan {
   std::vector<ParallelLayer> layers;
-  int width, vocab_rows, prefill_rows, out_cols_max, q_max;
+  RowsPlan rows;
+  int width, vocab_rows, out_cols_max, q_max;
   float embed_scale;
   const float *embed_norm, *final_norm;
   const double *turns;
@@ -81,11 +96,32 @@ struct ParallelPlan {
   /* of a portion of a prompt: rows_cap positions */
   float *rows_gate;
   void *rows_mixed_terms;
-  /* of the positions whose logits are asked for: want_cap of them */
-  int32_t *want;
-  void *want_terms;
-  float *want_logits;
-  int want_cap;
+};
+
+/* One run of a layer around a residual of several streams: its weights (a layer that
+   runs several times has them several times here) and where this run's ring or state
+   lies. */
+struct StreamLayer {
+  vx_stream_layer l;
+  int in_rows, out_cols, window, cache_rows;
+  int64_t at;           /* floats from k_cache to this run's ring or state */
+  int64_t batch_stride; /* floats from a sequence's ring or state to the next one's */
+};
+struct StreamPlan {
+  std::vector<StreamLayer> layers;
+  RowsPlan rows;
+  int width, vocab_rows, streams;
+  float embed_scale, logit_scale, logit_cap;
+  const float *final_norm;
+  int64_t cache_floats;
+  int in_max, q_max, q_rank_max, mixed_max, hidden_max;
+  /* of a step: [batch][in_max], [batch][q_max], [batch][mixed_max],
+     [batch][hidden_max], [batch][q_rank_max] */
+  float *in, *q, *mixed, *hidden, *q_latent;
+  /* of a portion of a prompt */
+  float *rows_q, *rows_alpha, *rows_o, *rows_kv;
+  void *rows_terms;
+  size_t q_floats, alpha_floats, o_floats, kv_floats, term_values;
 };
 
 struct vx_decoder {
@@ -142,6 +178,8 @@ struct vx_decoder {
   int logit_stride;
   /* a decoder of parallel blocks (decoder_parallel.cu), or NULL */
   ParallelPlan *par;
+  /* a decoder of layers around several streams (decoder_streams.cu), or NULL */
+  StreamPlan *streams;
 };
 
 /* decoder.cu: the tokens of a step (agreed between the ranks of a vocabulary-split
@@ -151,5 +189,14 @@ void decoder_advance(vx_decoder *d, int count);
 /* decoder_parallel.cu */
 void decoder_record_parallel_step(vx_decoder *d);
 void decoder_free_parallel(vx_decoder *d);
+/* The next t positions of the sequence through all layers, and the logits [n_want,
+   vocab] of the places `want` lists. */
+void decoder_parallel_rows(vx_decoder *d, const int32_t *tokens, int t,
+                           const int32_t *want, int n_want, float *logits);
+/* decoder_streams.cu: the same for its decoders */
+void decoder_record_stream_step(vx_decoder *d);
+void decoder_free_streams(vx_decoder *d);
+void decoder_stream_rows(vx_decoder *d, const int32_t *tokens, int t, const int32_t *want,
+                         int n_want, float *logits);
 
 #endif /* VXB_DECODER_STATE_H */

@@ -1,0 +1,483 @@
+/* gated_linear.cu -- gated linear attention: a matrix per head that fades by key
+ * channel, takes in k v^T and is read by q.
+ *
+ * A column of the state needs no other column, so both forms cut the state by
+ * columns.  A step streams it once (a cluster per head, so that the norm over the
+ * head meets in distributed shared memory).  The positions of a prompt go through
+ * one after another with the state in registers: 3 multiply-adds per value of the
+ * state and position, which is what a chunked form costs on the FP32 pipe too, and
+ * the result does not depend on how the prompt is cut.
+ */
+#include "kernels.h"
+#include "launch.cuh"
+#include "launch_util.h"
+#include "nn_device.cuh"
+#include "terms.cuh"
+
+#include <cooperative_groups.h>
+
+namespace vxb {
+namespace {
+
+namespace cg = cooperative_groups;
+
+/* sigmoid(z)^(1 / tau), by way of the logarithm, which no z overflows */
+__device__ __forceinline__ float decay(float z, float inv_tau) {
+  const float log_sigmoid = fminf(z, 0.0f) - log1pf(expf(-fabsf(z)));
+  return expf(log_sigmoid * inv_tau);
+}
+
+/* where the parts of an input row begin */
+struct Parts {
+  int k, v, gate, a1;
+  __host__ __device__ explicit Parts(const GatedLinearArgs &a)
+      : k(a.heads * a.dim), v(2 * k), gate(v + a.heads * a.vdim),
+        a1(gate + a.heads * a.vdim) {}
+};
+
+/* ---- one token of each sequence ------------------------------------------------
+ * A cluster of CL blocks per (head, sequence), block r taking vdim / CL columns
+ * (rounded up to 4). Threads: 8 groups of four columns by 32 rows. */
+constexpr int CL = 8, STEP_THREADS = 256, COLS4 = 8, ROWS = STEP_THREADS / COLS4;
+constexpr int EARLY = 8; /* rows of a thread that are fetched ahead of the wait */
+
+__global__ void __launch_bounds__(STEP_THREADS)
+gated_linear_step_kernel(const GatedLinearArgs a, const float *in, int64_t in_stride,
+                         float *out, int64_t out_stride) {
+  extern __shared__ __align__(16) float step_smem[];
+  const int slice4 = (a.vdim / 4 + CL - 1) / CL; /* float4 columns of a block */
+  float *alpha = step_smem, *sk = alpha + a.dim, *sq = sk + a.dim; /* [dim] each */
+  float *o = sq + a.dim;                                           /* [slice4 * 4] */
+  __shared__ __align__(16) float part[ROWS][COLS4 * 4 + 4];
+  __shared__ float ssq, red[STEP_THREADS / 32];
+  chain_release();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int h = blockIdx.y, b = blockIdx.z, r = blockIdx.x;
+  const int c4 = tid % COLS4, row = tid / COLS4;
+  const int first4 = r * slice4, last4 = min(first4 + slice4, a.vdim / 4);
+  const bool fresh = a.positions[b] == 0;
+  float *state = a.state + b * a.state_batch_stride + (int64_t)h * a.dim * a.vdim;
+  const Parts at(a);
+
+  /* The state is what earlier steps left: the first columns' rows come while the
+     kernel in front still runs. */
+  float4 early[EARLY];
+#pragma unroll
+  for (int j = 0; j < EARLY; ++j) {
+    const int i = row + j * ROWS;
+    early[j] = make_float4(0, 0, 0, 0);
+    if (!fresh && i < a.dim && first4 + c4 < last4)
+      early[j] = *reinterpret_cast<const float4 *>(state + (int64_t)i * a.vdim +
+                                                   (first4 + c4) * 4);
+  }
+  chain_wait();
+  const float *x = in + b * in_stride;
+  for (int i = tid; i < a.dim; i += STEP_THREADS) {
+    float z = a.a2_bias[h * a.dim + i];
+    const float4 *w = reinterpret_cast<const float4 *>(a.a2 +
+                                                       (int64_t)(h * a.dim + i) * a.rank);
+    const float4 *y = reinterpret_cast<const float4 *>(x + at.a1);
+    for (int c = 0; c < a.rank / 4; ++c) {
+      const float4 p = w[c], q = y[c];
+      z = fmaf(p.x, q.x, z);
+      z = fmaf(p.y, q.y, z);
+      z = fmaf(p.z, q.z, z);
+      z = fmaf(p.w, q.w, z);
+    }
+    alpha[i] = decay(z, a.inv_tau);
+    sk[i] = x[at.k + h * a.dim + i];
+    sq[i] = x[h * a.dim + i] * a.q_scale;
+  }
+  __syncthreads();
+
+  float ss = 0.0f;
+  for (int base4 = first4; base4 < last4; base4 += COLS4) {
+    const int col4 = base4 + c4;
+    const bool mine = col4 < last4;
+    float4 v = make_float4(0, 0, 0, 0), sum = v;
+    if (mine)
+      v = *reinterpret_cast<const float4 *>(x + at.v + h * a.vdim + col4 * 4);
+    auto advance = [&](int i, float4 s) {
+      const float f = alpha[i], k = sk[i];
+      s.x = fmaf(k, v.x, f * s.x);
+      s.y = fmaf(k, v.y, f * s.y);
+      s.z = fmaf(k, v.z, f * s.z);
+      s.w = fmaf(k, v.w, f * s.w);
+      *reinterpret_cast<float4 *>(state + (int64_t)i * a.vdim + col4 * 4) = s;
+      axpy(sum, sq[i], s);
+    };
+    if (mine) {
+      int i = row;
+      if (base4 == first4) {
+#pragma unroll
+        for (int j = 0; j < EARLY; ++j, i += ROWS)
+          if (i < a.dim)
+            advance(i, early[j]);
+      }
+      for (; i < a.dim; i += ROWS)
+        advance(i, fresh ? make_float4(0, 0, 0, 0)
+                         : *reinterpret_cast<const float4 *>(
+                               state + (int64_t)i * a.vdim + col4 * 4));
+    }
+    *reinterpret_cast<float4 *>(&part[row][c4 * 4]) = sum;
+    __syncthreads();
+    if (tid < COLS4 * 4 && (base4 - first4) * 4 + tid < slice4 * 4) {
+      float total = 0.0f;
+      for (int k = 0; k < ROWS; ++k) /* fixed order */
+        total += part[k][tid];
+      o[(base4 - first4) * 4 + tid] = total;
+      ss = fmaf(total, total, ss);
+    }
+    __syncthreads();
+  }
+  ss = warp_sum(ss);
+  if (lane == 0)
+    red[warp] = ss;
+  __syncthreads();
+  if (tid == 0) {
+    float total = 0.0f;
+    for (int k = 0; k < STEP_THREADS / 32; ++k)
+      total += red[k];
+    ssq = total;
+  }
+  cg::cluster_group cluster = cg::this_cluster();
+  cluster.sync();
+  float total = 0.0f;
+  for (int k = 0; k < CL; ++k) /* fixed order */
+    total += *cluster.map_shared_rank(&ssq, k);
+  const float inv = 1.0f / sqrtf(total / (float)a.v_mean + a.eps);
+  for (int c = tid; c < (last4 - first4) * 4; c += STEP_THREADS) {
+    const int col = first4 * 4 + c;
+    const float g = x[at.gate + h * a.vdim + col];
+    out[b * out_stride + h * a.vdim + col] = o[c] * inv * a.gain[col] * silu(g);
+  }
+  cluster.sync(); /* nobody leaves while a peer may still read its sum */
+}
+
+/* ---- the positions of a prompt: decays -----------------------------------------
+ * A block takes TB positions and 256 channels. */
+constexpr int TB = 16;
+__global__ void __launch_bounds__(256)
+gated_linear_decay_kernel(const GatedLinearArgs a, const float *in, int64_t in_stride,
+                          int t_count, float *alpha) {
+  extern __shared__ __align__(16) float low[]; /* [TB][rank] */
+  chain_release();
+  chain_wait();
+  const int t0 = blockIdx.x * TB, channels = a.heads * a.dim;
+  const int a1 = Parts(a).a1;
+  for (int i = threadIdx.x; i < TB * a.rank; i += 256) {
+    const int t = i / a.rank, c = i - t * a.rank;
+    low[i] = t0 + t < t_count ? in[(t0 + t) * in_stride + a1 + c] : 0.0f;
+  }
+  __syncthreads();
+  const int ch = blockIdx.y * 256 + threadIdx.x;
+  if (ch >= channels)
+    return;
+  float z[TB];
+  const float bias = a.a2_bias[ch];
+#pragma unroll
+  for (int t = 0; t < TB; ++t)
+    z[t] = bias;
+  const float4 *w = reinterpret_cast<const float4 *>(a.a2 + (int64_t)ch * a.rank);
+  for (int c = 0; c < a.rank / 4; ++c) {
+    const float4 p = w[c];
+#pragma unroll
+    for (int t = 0; t < TB; ++t) {
+      const float4 y = *reinterpret_cast<const float4 *>(&low[t * a.rank + c * 4]);
+      z[t] = fmaf(p.x, y.x, z[t]);
+      z[t] = fmaf(p.y, y.y, z[t]);
+      z[t] = fmaf(p.z, y.z, z[t]);
+      z[t] = fmaf(p.w, y.w, z[t]);
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < TB; ++t)
+    if (t0 + t < t_count)
+      alpha[(int64_t)(t0 + t) * channels + ch] = decay(z[t], a.inv_tau);
+}
+
+/* ---- the positions of a prompt: the recurrence ----------------------------------
+ * LG lanes side by side hold the key channels of RJ columns (lane g of them channels
+ * 4 (LG c + g) .. + 3, c below NI), so a warp holds 32 / LG * RJ columns of a head
+ * and a block SCAN_WARPS times as many. q, k, alpha and v of TT positions at a time
+ * come through two shared-memory buffers. Two columns go through a multiply-add
+ * together. */
+constexpr int SCAN_WARPS = 4, SCAN_THREADS = SCAN_WARPS * 32, TT = 16;
+
+__device__ __forceinline__ void copy16(float *dst, const float *src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(ptx::smem_addr(dst)),
+               "l"(src)
+               : "memory");
+}
+
+/* The sums over the LG lanes of a group: half of the values change hands at every
+   exchange while there are several. Returns the one that this lane is left with;
+   `col` says which it is, `owner` whether this lane is to write it. */
+template <int LG, int RJ>
+__device__ __forceinline__ float group_sums(float (&v)[RJ], int g, int &col, bool &owner) {
+  col = 0;
+  owner = true;
+  int off = LG / 2;
+#pragma unroll
+  for (int n = RJ; n > 1; n /= 2) {
+    const bool upper = (g & off) != 0;
+#pragma unroll
+    for (int j = 0; j < RJ / 2; ++j)
+      if (j < n / 2) {
+        const float give = upper ? v[j] : v[j + n / 2];
+        const float keep = upper ? v[j + n / 2] : v[j];
+        v[j] = keep + __shfl_xor_sync(0xffffffffu, give, off);
+      }
+    if (upper)
+      col += n / 2;
+    off /= 2;
+  }
+  float s = v[0];
+#pragma unroll
+  for (int rest = LG / 2 / RJ; rest > 0; rest /= 2) {
+    s += __shfl_xor_sync(0xffffffffu, s, rest);
+    owner = owner && (g & rest) == 0;
+  }
+  return s;
+}
+
+template <int LG, int NI, int RJ>
+__global__ void __launch_bounds__(SCAN_THREADS)
+gated_linear_scan_kernel(const GatedLinearArgs a, const float *in, int64_t in_stride,
+                         const float *alpha, int t_count, float *o) {
+  static_assert(LG >= RJ && RJ >= 2, "a group has a lane for every column");
+  constexpr int WARP_COLS = 32 / LG * RJ, COLS = SCAN_WARPS * WARP_COLS;
+  extern __shared__ __align__(16) float scan_smem[];
+  const int dim = a.dim, vdim = a.vdim;
+  const int step = 3 * dim + COLS; /* floats of a position: q | k | alpha | v */
+  float *buf = scan_smem;          /* [2][TT][step] */
+  float *so = buf + 2 * TT * step; /* [TT][COLS] */
+  chain_release();
+  chain_wait();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int h = blockIdx.y, col0 = blockIdx.x * COLS;
+  const int g = lane % LG, group = lane / LG;
+  const int mine = warp * WARP_COLS + group * RJ; /* first column, in the block */
+  const Parts at(a);
+  const bool fresh = a.positions[0] == 0;
+  float *state = a.state + (int64_t)h * dim * vdim;
+
+  auto fetch = [&](int t0, float *to) {
+    const int quads = step / 4, dq = dim / 4, n = min(TT, t_count - t0);
+    for (int i = tid; i < n * quads; i += SCAN_THREADS) {
+      const int t = i / quads, q = i - t * quads;
+      const float *row = in + (int64_t)(t0 + t) * in_stride;
+      float *dst = to + t * step + q * 4;
+      if (q < dq)
+        copy16(dst, row + h * dim + q * 4);
+      else if (q < 2 * dq)
+        copy16(dst, row + at.k + h * dim + (q - dq) * 4);
+      else if (q < 3 * dq)
+        copy16(dst, alpha + (int64_t)(t0 + t) * a.heads * dim + h * dim +
+                        (q - 2 * dq) * 4);
+      else if (col0 + (q - 3 * dq) * 4 < vdim)
+        copy16(dst, row + at.v + h * vdim + col0 + (q - 3 * dq) * 4);
+      else
+        *reinterpret_cast<float4 *>(dst) = make_float4(0, 0, 0, 0);
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  };
+
+  float2 s[4 * NI][RJ / 2];
+#pragma unroll
+  for (int c = 0; c < NI; ++c)
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+#pragma unroll
+      for (int j = 0; j < RJ / 2; ++j) {
+        const int i = (c * LG + g) * 4 + e, col = col0 + mine + 2 * j;
+        s[c * 4 + e][j] = make_float2(0, 0);
+        if (!fresh && i < dim && col < vdim)
+          s[c * 4 + e][j] =
+              *reinterpret_cast<const float2 *>(state + (int64_t)i * vdim + col);
+      }
+  fetch(0, buf);
+  int side = 0;
+  for (int t0 = 0; t0 < t_count; t0 += TT, side ^= 1) {
+    const int n = min(TT, t_count - t0);
+    if (t0 + TT < t_count) {
+      fetch(t0 + TT, buf + (side ^ 1) * TT * step);
+      asm volatile("cp.async.wait_group 1;" ::: "memory");
+    } else {
+      asm volatile("cp.async.wait_group 0;" ::: "memory");
+    }
+    __syncthreads();
+    const float *now = buf + side * TT * step;
+#pragma unroll 2
+    for (int t = 0; t < n; ++t, now += step) {
+      float2 v[RJ / 2], sum[RJ / 2];
+#pragma unroll
+      for (int j = 0; j < RJ / 2; ++j) {
+        v[j] = *reinterpret_cast<const float2 *>(now + 3 * dim + mine + 2 * j);
+        sum[j] = make_float2(0, 0);
+      }
+#pragma unroll
+      for (int c = 0; c < NI; ++c) {
+        const int i = (c * LG + g) * 4;
+        float4 q4 = make_float4(0, 0, 0, 0), k4 = q4, f4 = q4;
+        if (i < dim) {
+          q4 = *reinterpret_cast<const float4 *>(now + i);
+          k4 = *reinterpret_cast<const float4 *>(now + dim + i);
+          f4 = *reinterpret_cast<const float4 *>(now + 2 * dim + i);
+        }
+        const float q[4] = {q4.x, q4.y, q4.z, q4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w},
+                    f[4] = {f4.x, f4.y, f4.z, f4.w};
+#pragma unroll
+        for (int e = 0; e < 4; ++e)
+#pragma unroll
+          for (int j = 0; j < RJ / 2; ++j) {
+            float2 &cell = s[c * 4 + e][j];
+            cell = mul_pair(make_float2(f[e], f[e]), cell);
+            fma_pair(cell, make_float2(k[e], k[e]), v[j]);
+            fma_pair(sum[j], make_float2(q[e], q[e]), cell);
+          }
+      }
+      float part[RJ];
+#pragma unroll
+      for (int j = 0; j < RJ / 2; ++j) {
+        part[2 * j] = sum[j].x;
+        part[2 * j + 1] = sum[j].y;
+      }
+      int col;
+      bool owner;
+      const float total = group_sums<LG, RJ>(part, g, col, owner);
+      if (owner)
+        so[t * COLS + mine + col] = total * a.q_scale;
+    }
+    __syncthreads(); /* the buffer may be filled again; so is complete */
+    for (int i = tid; i < n * (COLS / 4); i += SCAN_THREADS) {
+      const int t = i / (COLS / 4), c = i % (COLS / 4) * 4;
+      if (col0 + c < vdim)
+        *reinterpret_cast<float4 *>(o + (int64_t)(t0 + t) * a.heads * vdim + h * vdim +
+                                    col0 + c) =
+            *reinterpret_cast<const float4 *>(&so[t * COLS + c]);
+    }
+  }
+#pragma unroll
+  for (int c = 0; c < NI; ++c)
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+#pragma unroll
+      for (int j = 0; j < RJ / 2; ++j) {
+        const int i = (c * LG + g) * 4 + e, col = col0 + mine + 2 * j;
+        if (i < dim && col < vdim)
+          *reinterpret_cast<float2 *>(state + (int64_t)i * vdim + col) = s[c * 4 + e][j];
+      }
+}
+
+/* ---- the positions of a prompt: norm and gate -----------------------------------
+ * A block is a position, a warp takes every eighth head. */
+__global__ void __launch_bounds__(256)
+gated_linear_finish_kernel(const GatedLinearArgs a, const float *in, int64_t in_stride,
+                           const float *o, __nv_bfloat16 *terms, int cols) {
+  chain_release();
+  chain_wait();
+  const int64_t t = blockIdx.x;
+  const int lane = threadIdx.x & 31, gate = Parts(a).gate;
+  for (int h = threadIdx.x >> 5; h < a.heads; h += 8) {
+    const float *row = o + (t * a.heads + h) * a.vdim;
+    const float *g = in + t * in_stride + gate + h * a.vdim;
+    float ss = 0.0f;
+    for (int c = lane * 4; c < a.vdim; c += 128) {
+      const float4 v = *reinterpret_cast<const float4 *>(row + c);
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(ss) / (float)a.v_mean + a.eps);
+    for (int c = lane * 4; c < a.vdim; c += 128) {
+      const float4 v = *reinterpret_cast<const float4 *>(row + c);
+      const float4 w = *reinterpret_cast<const float4 *>(a.gain + c);
+      const float4 z = *reinterpret_cast<const float4 *>(g + c);
+      const float out[4] = {v.x * inv * w.x * silu(z.x), v.y * inv * w.y * silu(z.y),
+                            v.z * inv * w.z * silu(z.z), v.w * inv * w.w * silu(z.w)};
+      store_terms4(terms, cols, t, h * a.vdim + c, out);
+    }
+  }
+}
+
+const char *refuse(const GatedLinearArgs &a, int64_t in_stride) {
+  if (a.heads < 1 || a.dim < 8 || a.dim > 512 || (a.dim | a.vdim | a.rank) % 8 != 0 ||
+      a.vdim < 8 || a.vdim > 16384 || a.rank < 8 || a.rank > 512)
+    return "gated linear attention takes head sizes and a rank in multiples of 8, keys "
+           "and rank at most 512";
+  if (in_stride % 4 != 0 || a.state_batch_stride % 4 != 0 ||
+      ((uintptr_t)a.state | (uintptr_t)a.a2 | (uintptr_t)a.gain) & 15)
+    return "the state and the rows of gated linear attention must be 16-byte aligned";
+  return nullptr;
+}
+
+template <int LG, int NI, int RJ>
+const char *launch_scan(const GatedLinearArgs &a, const float *in, int64_t in_stride,
+                        const float *alpha, int t, float *o, cudaStream_t stream) {
+  constexpr int COLS = SCAN_WARPS * 32 / LG * RJ;
+  const int smem = (2 * TT * (3 * a.dim + COLS) + TT * COLS) * (int)sizeof(float);
+  constexpr int most =
+      (2 * TT * (3 * LG * NI * 4 + COLS) + TT * COLS) * (int)sizeof(float);
+  static_assert(most <= 227 * 1024, "the buffers fit in shared memory");
+  const void *kernel = (const void *)gated_linear_scan_kernel<LG, NI, RJ>;
+  if (allow_dynamic_smem(kernel, most) != cudaSuccess)
+    return "gated linear attention could not get its shared memory";
+  launch_chained(gated_linear_scan_kernel<LG, NI, RJ>,
+                 dim3((a.vdim + COLS - 1) / COLS, a.heads), dim3(SCAN_THREADS), smem,
+                 stream, a, in, in_stride, alpha, t, o);
+  return check_launch("the recurrence of gated linear attention");
+}
+
+} // namespace
+
+const char *gated_linear_decode(const GatedLinearArgs &a, const float *in,
+                                int64_t in_stride, int batch, float *out,
+                                int64_t out_stride, cudaStream_t stream) {
+  if (const char *why = refuse(a, in_stride))
+    return why;
+  const int slice4 = (a.vdim / 4 + CL - 1) / CL;
+  const int smem = (3 * a.dim + slice4 * 4) * (int)sizeof(float);
+  launch_chained_cluster_smem(gated_linear_step_kernel, dim3(CL, a.heads, batch),
+                              dim3(STEP_THREADS), CL, smem, stream, a, in, in_stride, out,
+                              out_stride);
+  return check_launch("a step of gated linear attention");
+}
+
+const char *gated_linear_decays(const GatedLinearArgs &a, const float *in,
+                                int64_t in_stride, int t, float *alpha,
+                                cudaStream_t stream) {
+  if (const char *why = refuse(a, in_stride))
+    return why;
+  launch_chained(gated_linear_decay_kernel,
+                 dim3((t + TB - 1) / TB, (a.heads * a.dim + 255) / 256), dim3(256),
+                 TB * a.rank * sizeof(float), stream, a, in, in_stride, t, alpha);
+  return check_launch("the decays of gated linear attention");
+}
+
+const char *gated_linear_scan(const GatedLinearArgs &a, const float *in, int64_t in_stride,
+                              const float *alpha, int t, float *o, cudaStream_t stream) {
+  if (const char *why = refuse(a, in_stride))
+    return why;
+  if (a.dim <= 32)
+    return launch_scan<8, 1, 8>(a, in, in_stride, alpha, t, o, stream);
+  if (a.dim <= 64)
+    return launch_scan<16, 1, 8>(a, in, in_stride, alpha, t, o, stream);
+  if (a.dim <= 128)
+    return launch_scan<32, 1, 8>(a, in, in_stride, alpha, t, o, stream);
+  if (a.dim <= 256)
+    return launch_scan<32, 2, 8>(a, in, in_stride, alpha, t, o, stream);
+  return launch_scan<32, 4, 4>(a, in, in_stride, alpha, t, o, stream);
+}
+
+const char *gated_linear_finish(const GatedLinearArgs &a, const float *in,
+                                int64_t in_stride, const float *o, int t, void *terms,
+                                int cols, cudaStream_t stream) {
+  if (const char *why = refuse(a, in_stride))
+    return why;
+  if (cols % 4 != 0 || cols < a.heads * a.vdim)
+    return "the output has too few columns";
+  launch_chained(gated_linear_finish_kernel, dim3(t), dim3(256), 0, stream, a, in,
+                 in_stride, o, (__nv_bfloat16 *)terms, cols);
+  return check_launch("the norm and gate of gated linear attention");
+}
+
+} // namespace vxb

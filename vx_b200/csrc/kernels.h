@@ -208,6 +208,40 @@ struct FanArgs {
 };
 const char *fan_proj(const FanArgs &a, cudaStream_t stream);
 
+/* ---- a residual of several streams ---------------------------------------------
+ * Instead of one residual x there are `streams` of them, [batch][streams][dim].
+ * A sublayer reads their weighted sum u = sum_s in[s] x_s through an RMSNorm, and
+ * its output y goes back into all of them at once, x_t <- sum_s mix[s][t] x_s +
+ * out[t] y from the old x_s (mix is [from][to]). One stream with in = mix = out = 1
+ * is the ordinary residual.
+ *   kStreamsStore, kStreamsGelu, kStreamsLogits: y = f(W norm(u)), f being nothing,
+ *     the exact gelu, or cap * tanh(scale * . / cap) (cap 0: scale * .); x
+ *     [batch][streams][dim], in NULL: all ones; norm_w NULL: one stream that is
+ *     normalised already.
+ *   kStreamsMix: y [batch][streams][dim] holds the streams, x is the sublayer's
+ *     input to its last matrix. */
+constexpr int kMaxStreams = 32;
+enum { kStreamsStore = 0, kStreamsGelu = 1, kStreamsLogits = 2, kStreamsMix = 3 };
+struct StreamProj {
+  int mode;
+  const void *w;
+  int fmt; /* kFmtF32 or kFmtBf16 */
+  int rows, cols;
+  const float *x;
+  int64_t x_stride;
+  int batch;
+  int streams;
+  int64_t stream_stride; /* values from one stream of a sequence to the next */
+  const float *in, *mix, *out;
+  const float *norm_w;
+  int norm_n;
+  float eps;
+  float *y;
+  int64_t y_stride;
+  float logit_scale, logit_cap;
+};
+const char *stream_proj(const StreamProj &a, cudaStream_t stream);
+
 /* The unfused pieces, for the operator surface. */
 const char *rope_and_store(float *q_out, float *k_cache, float *v_cache,
                            const float *q, const float *k, const float *v,
@@ -418,7 +452,8 @@ int rows_status();
 /* ---- what a parallel block needs besides (parallel_block.cu, window_attention.cu)
  * Token rows into the residual: scale * table[token], plus the sinusoid of the
  * position (sin at 2i, cos at 2i + 1; turns[i], f64: how much of a full turn the
- * pair's angle advances per position), through an RMSNorm. Rows are `dim`
+ * pair's angle advances per position; NULL: no sinusoid), through an RMSNorm
+ * (gain NULL: none), into `copies` rows one after another. Rows are `dim`
  * values of which `width` are the model's and the rest zeros. per_sequence:
  * row b is sequence b at positions[b]; else row t is at positions[0] + t. A token
  * outside the table gives a row of NaN. */
@@ -434,6 +469,7 @@ struct PositionEmbedArgs {
   float eps;
   const int32_t *positions;
   bool per_sequence;
+  int copies; /* 0: one */
 };
 const char *position_embed(const PositionEmbedArgs &a, cudaStream_t stream);
 
@@ -472,9 +508,118 @@ const char *rows_fan_finish(const float *partials, int splits, int t, int n,
    sum of its three terms. One run. cols a multiple of 16. */
 const char *rows_gemm_f32(const void *terms, const float *w, int t, int n, int cols,
                           float *partials, cudaStream_t stream);
-/* out[t][r] = the runs' sum, r below n. */
+/* out[t][r] = the runs' sum, r below n (out may be the partials); times `scale`
+   and then, with `cap` above 0, capped: cap * tanh(. / cap). */
 const char *rows_sum(float *out, const float *partials, int splits, int t, int n,
-                     cudaStream_t stream);
+                     cudaStream_t stream, float scale = 1.0f, float cap = 0.0f);
+
+/* ---- a residual of several streams, many positions (residual_streams.cu) --------
+ * x [t][streams][dim]. How a sublayer reads the streams and writes them (see
+ * StreamProj); in NULL: all ones. */
+struct StreamMix {
+  int streams;
+  const float *in, *mix, *out;
+};
+/* Terms of RMSNorm(sum_s in[s] x_s) * w of t positions (of those `pick` lists). */
+const char *rows_streams_norm(void *terms, const float *x, const StreamMix &m, NormGain w,
+                              int t, int dim, float eps, cudaStream_t stream,
+                              const int32_t *pick = nullptr);
+/* The same as f32 rows y[batch][dim], for steps whose sequences do not fit the
+   projections' shared memory; x_stride: values from one sequence's streams to the
+   next one's. */
+const char *streams_norm(float *y, const float *x, int64_t x_stride, const StreamMix &m,
+                         NormGain w, int batch, int dim, float eps, cudaStream_t stream);
+/* x_t <- sum_s mix[s][t] x_s + out[t] (the product), then, unless terms is NULL,
+   the terms of the next sublayer's norm (its in and w). */
+const char *rows_streams_mix(void *terms, float *x, const float *partials, int splits,
+                             int t, const StreamMix &m, const float *next_in, NormGain w,
+                             int dim, float eps, cudaStream_t stream);
+/* Terms of gelu(the product), hidden a multiple of 8. */
+const char *rows_gelu_finish(void *terms, const float *partials, int splits, int t,
+                             int hidden, cudaStream_t stream);
+
+/* ---- latent attention (latent_attention.cu) -------------------------------------
+ * Keys and values of all heads are products of one latent c per position, and a
+ * rotated key part is shared by the heads, so a ring of [kv_rank | rot] f32 rows
+ * (position t in row t % cache_rows) is the whole cache. The score of head h is
+ * scale * (q_h . W_uk_h c + q'_h . k'), the value W_uv_h c; a token at p sees
+ * p - window + 1 .. p. dim, rot, vdim: multiples of 8; kv_rank: of 64; what fills
+ * sizes up is zero. The pairs (2i, 2i + 1) of the rotated parts turn by turns[i] of a
+ * full turn per position. */
+struct LatentArgs {
+  int heads, dim, rot, vdim, kv_rank;
+  int window, cache_rows;
+  float scale;
+  float *ring;
+  int64_t ring_batch_stride;
+  const float *gain; /* of the latent's norm, over kv_mean values */
+  int kv_mean;
+  float eps;
+  const double *turns;
+  const int32_t *positions;
+  /* matrices in format `fmt`: w_ukv [heads][dim key rows, vdim value rows][kv_rank],
+     and the key rows of each head transposed, w_uk_t [heads][kv_rank][dim] */
+  const void *w_ukv, *w_uk_t;
+  int fmt;
+};
+/* A new token of each sequence: q [batch][heads][dim | rot] not rotated yet, down
+   [batch][down_stride] holding its [kv_rank | rot] before norm and rotation; puts
+   its row into the ring and the heads' values [heads][vdim] into out. The queries
+   go through W_uk and the weighted latents through W_uv inside the kernel, and no
+   key or value is ever made. cache_rows >= window. Rows below the position were
+   written before the chain of dependent launches began. */
+const char *latent_attention_decode(const LatentArgs &a, const float *q, int64_t q_stride,
+                                    const float *down, int64_t down_stride, int batch,
+                                    float *out, int64_t out_stride, cudaStream_t stream);
+/* After the product with rows [q_rank | kv_rank | rot]: the normalised query latent
+   as terms [t][3 q_rank], the ring's rows of the t positions. */
+const char *latent_rows_down(const LatentArgs &a, const float *partials, int splits, int t,
+                             int q_rank, const float *q_gain, int q_mean, void *terms,
+                             cudaStream_t stream);
+/* After the query product: q [t][heads][dim | rot], rotated. */
+const char *latent_rows_q(const LatentArgs &a, const float *partials, int splits, int t,
+                          float *q, cudaStream_t stream);
+/* Terms [n][3 kv_rank] of the latents of positions first .. first + n - 1. */
+const char *latent_rows_gather(const LatentArgs &a, int first, int n, void *terms,
+                               cudaStream_t stream);
+/* t positions of one sequence over keys and values that were made for the positions
+   from `first` on, kv [.][heads][dim | vdim] (the rotated part comes from the ring);
+   the output as terms in the first columns of [t][3 cols]. */
+const char *latent_attention_rows(const LatentArgs &a, const float *q, const float *kv,
+                                  int first, int t, void *terms, int cols,
+                                  cudaStream_t stream);
+
+/* ---- gated linear attention (gated_linear.cu) ------------------------------------
+ * Per head a state S [dim][vdim]: S <- diag(alpha) S + k v^T, o = S^T q, with a decay
+ * alpha = sigmoid(W_a2 a1 + bias)^(1 / tau) per key channel; then an RMSNorm of o over
+ * the head and silu(gate). A row of `in` is q | k | v | gate | a1, heads side by side;
+ * dim, vdim and a1's rank are multiples of 8, filled up with zeros. All of it f32; a
+ * sequence at position 0 starts from zero whatever its state holds. */
+struct GatedLinearArgs {
+  int heads, dim, vdim, rank;
+  float q_scale, inv_tau, eps;
+  int v_mean;            /* values of a head the norm's mean is over */
+  const float *a2, *a2_bias; /* [heads * dim][rank], [heads * dim] */
+  const float *gain;     /* [vdim] */
+  float *state;          /* [batch][heads][dim][vdim] */
+  int64_t state_batch_stride;
+  const int32_t *positions;
+};
+/* One token of each sequence: out [batch][out_stride]. */
+const char *gated_linear_decode(const GatedLinearArgs &a, const float *in,
+                                int64_t in_stride, int batch, float *out,
+                                int64_t out_stride, cudaStream_t stream);
+/* t positions of one sequence, in [t][in_stride]: alpha [t][heads * dim], then o
+   [t][heads * vdim] and the state after the last of them. */
+const char *gated_linear_decays(const GatedLinearArgs &a, const float *in,
+                                int64_t in_stride, int t, float *alpha,
+                                cudaStream_t stream);
+const char *gated_linear_scan(const GatedLinearArgs &a, const float *in, int64_t in_stride,
+                              const float *alpha, int t, float *o, cudaStream_t stream);
+/* Norm and gate of o, as terms in the first columns of [t][3 cols]. */
+const char *gated_linear_finish(const GatedLinearArgs &a, const float *in,
+                                int64_t in_stride, const float *o, int t, void *terms,
+                                int cols, cudaStream_t stream);
 
 /* nn_top_k (nn.vx:904-938): ids[j] = the index of the j-th largest of the
    first n logits (n <= 256; of equal values the lower index first), weights[j]

@@ -1,0 +1,794 @@
+/* latent_attention.cu -- attention whose keys and values are products of one latent
+ * per position, over a sliding window of a ring of latents.
+ *
+ * A step never makes a key or a value: a head's query goes through its key matrix
+ * once (q W_uk is a query for the latents themselves), the softmax weighs latents, and
+ * the sum goes through the head's value matrix; both products happen in the attention
+ * kernel, split over the blocks of a cluster.  All heads read one row per position, so
+ * a step moves kv_rank + rot values per position instead of heads * (dim + vdim).
+ * Over the positions of a prompt the latents are worth expanding: keys and values of
+ * the window are made by one GEMM, and a score costs dim + rot multiplications, not
+ * kv_rank + rot.  Scores, weights and sums are f32.
+ */
+#include "kernels.h"
+#include "launch.cuh"
+#include "launch_util.h"
+#include "nn_device.cuh"
+#include "terms.cuh"
+
+#include <cooperative_groups.h>
+
+namespace vxb {
+namespace {
+
+namespace cg = cooperative_groups;
+
+constexpr float LOWEST = -3.0e38f;
+
+/* ---- one new token per sequence ----------------------------------------------
+ * A cluster of CL blocks per (sequence, tile of GH heads); block r takes the r-th run
+ * of the window's positions and the r-th part of the two products' rows, its NW warps
+ * every NW-th position, NB rows of the ring in flight per warp. A lane holds D4
+ * float4s of a row. Warps and blocks meet in a fixed order. */
+constexpr int CL = 8;
+
+/* floats of dynamic shared memory */
+constexpr int latent_smem(int GH, int D4, int NW, int dim, int kv_rank) {
+  return (NW * GH + GH + 1) * D4 * 128 + GH * dim + GH * kv_rank / CL;
+}
+
+__device__ __forceinline__ float dot_word(const uint4 &w, const float *x,
+                                          const __nv_bfloat16 *) {
+  const float4 a = *reinterpret_cast<const float4 *>(x);
+  const float4 b = *reinterpret_cast<const float4 *>(x + 4);
+  float s = bf_lo(w.x) * a.x;
+  s = fmaf(bf_hi(w.x), a.y, s);
+  s = fmaf(bf_lo(w.y), a.z, s);
+  s = fmaf(bf_hi(w.y), a.w, s);
+  s = fmaf(bf_lo(w.z), b.x, s);
+  s = fmaf(bf_hi(w.z), b.y, s);
+  s = fmaf(bf_lo(w.w), b.z, s);
+  return fmaf(bf_hi(w.w), b.w, s);
+}
+__device__ __forceinline__ float dot_word(const uint4 &w, const float *x, const float *) {
+  const float4 a = *reinterpret_cast<const float4 *>(x);
+  float s = __uint_as_float(w.x) * a.x;
+  s = fmaf(__uint_as_float(w.y), a.y, s);
+  s = fmaf(__uint_as_float(w.z), a.z, s);
+  return fmaf(__uint_as_float(w.w), a.w, s);
+}
+
+/* `tasks` dot products of `cols` values by a block's warps: row(i) is the weights of
+   task i, in(i) its input in shared memory, put(i, s) takes the result. As many lanes
+   as a row has words take one, U tasks of each such group are in flight. */
+template <typename W, int NW, typename Row, typename In, typename Put>
+__device__ __forceinline__ void block_dots(int tasks, int cols, Row row, In in, Put put) {
+  constexpr int E = 16 / (int)sizeof(W), U = 4;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int words = cols / E;
+  int lanes = 32;
+  while (lanes > 1 && lanes / 2 >= words)
+    lanes /= 2;
+  const int groups = 32 / lanes, group = lane / lanes, first = lane % lanes;
+  for (int t0 = warp * groups * U; t0 < tasks; t0 += NW * groups * U) {
+    float s[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u)
+      s[u] = 0.0f;
+#pragma unroll 2
+    for (int wd = first; wd < words; wd += lanes) {
+      uint4 w[U];
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int i = t0 + u * groups + group;
+        w[u] = make_uint4(0, 0, 0, 0);
+        if (i < tasks)
+          w[u] = __ldg(reinterpret_cast<const uint4 *>(row(i)) + wd);
+      }
+#pragma unroll
+      for (int u = 0; u < U; ++u) {
+        const int i = t0 + u * groups + group;
+        if (i < tasks)
+          s[u] += dot_word(w[u], in(i) + wd * E, (const W *)nullptr);
+      }
+    }
+    for (int o = lanes / 2; o > 0; o >>= 1)
+#pragma unroll
+      for (int u = 0; u < U; ++u)
+        s[u] += __shfl_xor_sync(0xffffffffu, s[u], o);
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = t0 + u * groups + group;
+      if (first == 0 && i < tasks)
+        put(i, s[u]);
+    }
+  }
+}
+
+template <typename W, int GH, int D4, int NW>
+__global__ void __launch_bounds__(NW * 32)
+latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
+                     const float *down, int64_t down_stride, float *out,
+                     int64_t out_stride) {
+  constexpr int NB = D4 == 1 ? 8 : D4 == 2 ? 4 : D4 <= 5 ? 2 : 1;
+  constexpr int THREADS = NW * 32, ROW = D4 * 128;
+  extern __shared__ __align__(16) float latent_shared[];
+  float *acc_s = latent_shared;         /* [NW][GH][ROW] */
+  float *heads_s = acc_s + NW * GH * ROW; /* [GH][ROW]: queries, then weighted latents */
+  float *fresh = heads_s + GH * ROW;    /* [ROW]: this position's row */
+  float *qn = fresh + ROW;              /* [GH][dim] */
+  float *slice = qn + GH * a.dim;       /* [GH][kv_rank / CL] */
+  __shared__ float warp_m[NW][GH], warp_l[NW][GH], red[NW];
+  __shared__ float block_m[GH], block_l[GH], share[GH][CL];
+  cg::cluster_group cluster = cg::this_cluster();
+  chain_release();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int rank = blockIdx.x, h0 = blockIdx.y * GH, b = blockIdx.z;
+  const int nh = min(GH, a.heads - h0);
+  const int K = a.kv_rank, part = K / CL, row_floats = K + a.rot;
+  const int v_part = (a.vdim + CL - 1) / CL, v0 = min(rank * v_part, a.vdim),
+            vn = min(v_part, a.vdim - v0);
+  const W *uk = (const W *)a.w_uk_t, *ukv = (const W *)a.w_ukv;
+  auto uk_row = [&](int g, int r) {
+    return uk + ((int64_t)(h0 + g) * K + rank * part + r) * a.dim;
+  };
+  auto uv_row = [&](int g, int r) {
+    return ukv + ((int64_t)(h0 + g) * (a.dim + a.vdim) + a.dim + v0 + r) * K;
+  };
+  /* what depends on no kernel before: the matrices on their way to L2 */
+  if (tid < nh) {
+    ptx::bulk_prefetch_l2(uk_row(tid, 0), part * a.dim * (int)sizeof(W));
+    if (vn > 0)
+      ptx::bulk_prefetch_l2(uv_row(tid, 0), vn * K * (int)sizeof(W));
+  }
+  const int pos = a.positions[b];
+  const int low = max(0, pos - a.window + 1);
+  const int run = (pos - low + CL) / CL; /* ceil of the count over CL */
+  const int t_begin = low + rank * run, t_end = min(t_begin + run, pos + 1);
+  const int row_low = low % a.cache_rows;
+  float *ring = a.ring + b * a.ring_batch_stride;
+  bool active[D4];
+#pragma unroll
+  for (int c = 0; c < D4; ++c)
+    active[c] = (c * 32 + lane) * 4 < row_floats;
+
+  /* Rows below pos come from earlier steps; row pos is made here. */
+  float4 kv[NB][D4];
+  auto load = [&](int t0, bool own) {
+#pragma unroll
+    for (int j = 0; j < NB; ++j) {
+      const int t = t0 + j * NW;
+      if (t >= t_end || (t == pos) != own)
+        continue;
+      int row = row_low + (t - low);
+      if (row >= a.cache_rows)
+        row -= a.cache_rows;
+      const float *src = own ? fresh : ring + (int64_t)row * row_floats;
+#pragma unroll
+      for (int c = 0; c < D4; ++c)
+        if (active[c])
+          kv[j][c] = *reinterpret_cast<const float4 *>(src + (c * 32 + lane) * 4);
+    }
+  };
+#pragma unroll
+  for (int j = 0; j < NB; ++j)
+#pragma unroll
+    for (int c = 0; c < D4; ++c)
+      kv[j][c] = make_float4(0, 0, 0, 0);
+  load(t_begin + warp, false);
+  chain_wait();
+
+  /* ---- this position's row; the queries, rotated ---- */
+  const float *dn = down + b * down_stride;
+  const float *q = q_in + b * q_stride + (int64_t)h0 * (a.dim + a.rot);
+  float ss = 0.0f;
+  for (int i = tid; i < K; i += THREADS) {
+    const float v = dn[i];
+    fresh[i] = v;
+    ss = fmaf(v, v, ss);
+  }
+  ss = warp_sum(ss);
+  if (lane == 0)
+    red[warp] = ss;
+  for (int i = tid; i < nh * a.dim; i += THREADS) {
+    const int g = i / a.dim;
+    qn[i] = q[g * (a.dim + a.rot) + i - g * a.dim];
+  }
+  const int pairs = a.rot / 2;
+  for (int i = tid; i < (nh + 1) * pairs; i += THREADS) {
+    const int g = i / pairs, k = i - g * pairs; /* g == nh: the key */
+    const float2 uv = *reinterpret_cast<const float2 *>(
+        (g < nh ? q + g * (a.dim + a.rot) + a.dim : dn + K) + 2 * k);
+    float sine, cosine;
+    turned(pos, a.turns[k], sine, cosine);
+    float *to = (g < nh ? heads_s + g * ROW : fresh) + K + 2 * k;
+    to[0] = uv.x * cosine - uv.y * sine;
+    to[1] = uv.y * cosine + uv.x * sine;
+  }
+  __syncthreads();
+  float total = 0.0f;
+  for (int w = 0; w < NW; ++w) /* fixed order */
+    total += red[w];
+  const float inv = 1.0f / sqrtf(total / (float)a.kv_mean + a.eps);
+  for (int i = tid; i < K; i += THREADS)
+    fresh[i] = fresh[i] * inv * a.gain[i];
+
+  /* ---- the queries for latents: this block's part of each, then all parts ---- */
+  block_dots<W, NW>(
+      nh * part, a.dim, [&](int i) { return uk_row(i / part, i % part); },
+      [&](int i) { return qn + i / part * a.dim; },
+      [&](int i, float s) { slice[i] = s; });
+  auto gather = [&] {
+    for (int i = tid; i < nh * K / 4; i += THREADS) {
+      const int g = i / (K / 4), c = (i - g * (K / 4)) * 4, r = c / part;
+      *reinterpret_cast<float4 *>(heads_s + g * ROW + c) =
+          *reinterpret_cast<const float4 *>(cluster.map_shared_rank(slice, r) +
+                                            g * part + c - r * part);
+    }
+  };
+  cluster.sync();
+  gather();
+  __syncthreads();
+  if (blockIdx.y == 0 && rank == 0) {
+    float *to = ring + (int64_t)(pos % a.cache_rows) * row_floats;
+    for (int i = tid; i < row_floats; i += THREADS)
+      to[i] = fresh[i];
+  }
+  load(t_begin + warp, true);
+
+  float4 qr[GH][D4], acc[GH][D4];
+  float m[GH], l[GH];
+#pragma unroll
+  for (int h = 0; h < GH; ++h) {
+    m[h] = LOWEST;
+    l[h] = 0.0f;
+#pragma unroll
+    for (int c = 0; c < D4; ++c) {
+      acc[h][c] = qr[h][c] = make_float4(0, 0, 0, 0);
+      if (active[c] && h < nh)
+        qr[h][c] =
+            *reinterpret_cast<const float4 *>(heads_s + h * ROW + (c * 32 + lane) * 4);
+    }
+  }
+  for (int t0 = t_begin + warp; t0 < t_end; t0 += NB * NW) {
+    if (t0 != t_begin + warp) {
+      load(t0, false);
+      load(t0, true);
+    }
+#pragma unroll
+    for (int h = 0; h < GH; ++h) {
+      float s[NB];
+#pragma unroll
+      for (int j = 0; j < NB; ++j) {
+        s[j] = 0.0f;
+#pragma unroll
+        for (int c = 0; c < D4; ++c) {
+          s[j] = fmaf(qr[h][c].x, kv[j][c].x, s[j]);
+          s[j] = fmaf(qr[h][c].y, kv[j][c].y, s[j]);
+          s[j] = fmaf(qr[h][c].z, kv[j][c].z, s[j]);
+          s[j] = fmaf(qr[h][c].w, kv[j][c].w, s[j]);
+        }
+      }
+#pragma unroll
+      for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+        for (int j = 0; j < NB; ++j)
+          s[j] += __shfl_xor_sync(0xffffffffu, s[j], o);
+      float big = m[h];
+#pragma unroll
+      for (int j = 0; j < NB; ++j) {
+        s[j] = t0 + j * NW < t_end ? s[j] * a.scale : LOWEST;
+        big = fmaxf(big, s[j]);
+      }
+      const float fix = expf(m[h] - big);
+      m[h] = big;
+      l[h] *= fix;
+#pragma unroll
+      for (int c = 0; c < D4; ++c) {
+        acc[h][c].x *= fix; acc[h][c].y *= fix;
+        acc[h][c].z *= fix; acc[h][c].w *= fix;
+      }
+#pragma unroll
+      for (int j = 0; j < NB; ++j) {
+        const float w = t0 + j * NW < t_end ? expf(s[j] - big) : 0.0f;
+        l[h] += w;
+#pragma unroll
+        for (int c = 0; c < D4; ++c)
+          axpy(acc[h][c], w, kv[j][c]);
+      }
+    }
+  }
+
+  /* ---- the block's warps, in warp order, into row 0 of its arrays ---- */
+#pragma unroll
+  for (int h = 0; h < GH; ++h) {
+    if (lane == 0) {
+      warp_m[warp][h] = m[h];
+      warp_l[warp][h] = l[h];
+    }
+#pragma unroll
+    for (int c = 0; c < D4; ++c)
+      *reinterpret_cast<float4 *>(acc_s + (warp * GH + h) * ROW + (c * 32 + lane) * 4) =
+          acc[h][c];
+  }
+  __syncthreads();
+  for (int i = warp; i < nh * D4; i += NW) {
+    const int h = i / D4, c = i - h * D4;
+    float big = LOWEST;
+    for (int w = 0; w < NW; ++w)
+      big = fmaxf(big, warp_m[w][h]);
+    float sum = 0.0f;
+    float4 o = make_float4(0, 0, 0, 0);
+    for (int w = 0; w < NW; ++w) {
+      const float f = expf(warp_m[w][h] - big);
+      sum = fmaf(f, warp_l[w][h], sum);
+      axpy(o, f,
+           *reinterpret_cast<const float4 *>(acc_s + (w * GH + h) * ROW +
+                                             (c * 32 + lane) * 4));
+    }
+    *reinterpret_cast<float4 *>(acc_s + h * ROW + (c * 32 + lane) * 4) = o;
+    if (lane == 0 && c == 0) {
+      block_m[h] = big;
+      block_l[h] = sum;
+    }
+  }
+
+  /* ---- the runs, in order: each block its part of the latents, then all parts ---- */
+  cluster.sync();
+  if (tid < nh) {
+    float pm[CL], big = LOWEST, sum = 0.0f;
+#pragma unroll
+    for (int r = 0; r < CL; ++r) {
+      pm[r] = cluster.map_shared_rank(block_m, r)[tid];
+      big = fmaxf(big, pm[r]);
+    }
+#pragma unroll
+    for (int r = 0; r < CL; ++r) {
+      pm[r] = expf(pm[r] - big);
+      sum = fmaf(pm[r], cluster.map_shared_rank(block_l, r)[tid], sum);
+    }
+#pragma unroll
+    for (int r = 0; r < CL; ++r)
+      share[tid][r] = pm[r] / sum;
+  }
+  __syncthreads();
+  for (int i = tid; i < nh * part / 4; i += THREADS) {
+    const int g = i / (part / 4), c = (i - g * (part / 4)) * 4;
+    float4 o = make_float4(0, 0, 0, 0);
+#pragma unroll
+    for (int r = 0; r < CL; ++r)
+      axpy(o, share[g][r],
+           *reinterpret_cast<const float4 *>(cluster.map_shared_rank(acc_s, r) + g * ROW +
+                                             rank * part + c));
+    *reinterpret_cast<float4 *>(slice + g * part + c) = o;
+  }
+  cluster.sync();
+  gather();
+  cluster.barrier_arrive(); /* nobody leaves while a peer may still read its part */
+  __syncthreads();
+
+  /* ---- through the value matrix ---- */
+  if (vn > 0)
+    block_dots<W, NW>(
+        nh * vn, K, [&](int i) { return uv_row(i / vn, i % vn); },
+        [&](int i) { return heads_s + i / vn * ROW; },
+        [&](int i, float s) {
+          out[b * out_stride + (int64_t)(h0 + i / vn) * a.vdim + v0 + i % vn] = s;
+        });
+  cluster.barrier_wait();
+}
+
+/* ---- the positions of a prompt: the ring's rows and the query latent -------------
+ * A block is a position. */
+__global__ void __launch_bounds__(256)
+latent_down_kernel(const LatentArgs a, const float *partials, int splits, int t_count,
+                   int q_rank, const float *q_gain, int q_mean, __nv_bfloat16 *terms) {
+  extern __shared__ float down_row[]; /* [q_rank + kv_rank] */
+  __shared__ float red[2][8];
+  chain_release();
+  chain_wait();
+  const int64_t t = blockIdx.x;
+  const int tid = threadIdx.x, K = a.kv_rank, both = q_rank + K, n = both + a.rot;
+  const int pos = a.positions[0] + (int)t;
+  float *ring = a.ring + (int64_t)(pos % a.cache_rows) * (K + a.rot);
+  float sq = 0.0f, sk = 0.0f;
+  for (int i = tid; i < both; i += 256) {
+    const float v = sum_runs(partials, splits, t_count, n, t, i);
+    down_row[i] = v;
+    if (i < q_rank)
+      sq = fmaf(v, v, sq);
+    else
+      sk = fmaf(v, v, sk);
+  }
+  sq = warp_sum(sq);
+  sk = warp_sum(sk);
+  if ((tid & 31) == 0) {
+    red[0][tid >> 5] = sq;
+    red[1][tid >> 5] = sk;
+  }
+  for (int k = tid; k < a.rot / 2; k += 256) {
+    const float u = sum_runs(partials, splits, t_count, n, t, both + 2 * k);
+    const float v = sum_runs(partials, splits, t_count, n, t, both + 2 * k + 1);
+    float sine, cosine;
+    turned(pos, a.turns[k], sine, cosine);
+    ring[K + 2 * k] = u * cosine - v * sine;
+    ring[K + 2 * k + 1] = v * cosine + u * sine;
+  }
+  __syncthreads();
+  sq = sk = 0.0f;
+  for (int w = 0; w < 8; ++w) { /* fixed order */
+    sq += red[0][w];
+    sk += red[1][w];
+  }
+  const float q_inv = 1.0f / sqrtf(sq / (float)q_mean + a.eps);
+  const float k_inv = 1.0f / sqrtf(sk / (float)a.kv_mean + a.eps);
+  for (int i = tid; i < both; i += 256) {
+    if (i < q_rank)
+      store_terms(terms, q_rank, t, i, down_row[i] * q_inv * q_gain[i]);
+    else
+      ring[i - q_rank] = down_row[i] * k_inv * a.gain[i - q_rank];
+  }
+}
+
+/* a thread per (position, four values of a head) */
+__global__ void __launch_bounds__(256)
+latent_q_kernel(const LatentArgs a, const float *partials, int splits, int t_count,
+                float *q) {
+  chain_release();
+  chain_wait();
+  const int hd = a.dim + a.rot, n = a.heads * hd;
+  const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= (int64_t)t_count * (n / 4))
+    return;
+  const int64_t t = idx / (n / 4);
+  const int r = (int)(idx - t * (n / 4)) * 4, d = r % hd;
+  float4 v = sum_runs4(partials, splits, t_count, n, t, r);
+  if (d >= a.dim) {
+    const int pos = a.positions[0] + (int)t, k = (d - a.dim) / 2;
+    float s0, c0, s1, c1;
+    turned(pos, a.turns[k], s0, c0);
+    turned(pos, a.turns[k + 1], s1, c1);
+    v = make_float4(v.x * c0 - v.y * s0, v.y * c0 + v.x * s0, v.z * c1 - v.w * s1,
+                    v.w * c1 + v.z * s1);
+  }
+  *reinterpret_cast<float4 *>(q + t * n + r) = v;
+}
+
+/* a thread per (position, eight values of its latent) */
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const LatentArgs a, int first, int n, __nv_bfloat16 *terms) {
+  chain_release();
+  chain_wait();
+  const int per_row = a.kv_rank / 8;
+  const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
+  if (idx >= (int64_t)n * per_row)
+    return;
+  const int64_t t = idx / per_row;
+  const int c = (int)(idx - t * per_row) * 8;
+  const float *row =
+      a.ring + (first + t) % a.cache_rows * (int64_t)(a.kv_rank + a.rot) + c;
+  const float4 lo = *reinterpret_cast<const float4 *>(row);
+  const float4 hi = *reinterpret_cast<const float4 *>(row + 4);
+  const float v[8] = {lo.x, lo.y, lo.z, lo.w, hi.x, hi.y, hi.z, hi.w};
+  store_terms8(terms, a.kv_rank, t, c, v);
+}
+
+/* ---- the positions of a prompt: attention -----------------------------------------
+ * A block per (AQ positions, head): scores against AK keys at a time, online softmax,
+ * weighted sum; 16 x 16 threads, thread (ty, tx) owning AQ / 16 queries, keys
+ * tx + 16 j and values tx * 4 + 64 c ... KP, VP: key and value sizes rounded up to
+ * what the threads cover, zeros beyond them. Two neighbouring values go through a
+ * multiply-add together. */
+constexpr int ROW_THREADS = 256;
+constexpr int rows_smem(int KP, int VP, int AQ, int AK) {
+  return ((AQ + AK) * (KP + 4) + AK * (VP + 4) + AQ * (AK + 4)) * 4;
+}
+
+template <int KP, int VP, int AQ, int AK>
+__global__ void __launch_bounds__(ROW_THREADS)
+latent_rows_kernel(const LatentArgs a, const float *q, const float *kv, int first,
+                   int t_count, __nv_bfloat16 *terms, int cols) {
+  constexpr int QN = AQ / 16, KN = AK / 16, CN = VP / 64;
+  extern __shared__ __align__(16) float att_smem[];
+  float (*sq)[KP + 4] = reinterpret_cast<float (*)[KP + 4]>(att_smem);
+  float (*sk)[KP + 4] = sq + AQ;
+  float (*sv)[VP + 4] = reinterpret_cast<float (*)[VP + 4]>(sk + AK);
+  float (*sp)[AK + 4] = reinterpret_cast<float (*)[AK + 4]>(sv + AK);
+  chain_release();
+  chain_wait();
+  const int dim = a.dim, hd = a.dim + a.rot, vdim = a.vdim, head = blockIdx.y;
+  const int t0 = blockIdx.x * AQ, base = a.positions[0];
+  const int tid = threadIdx.x, ty = tid / 16, tx = tid % 16;
+  const int row_floats = a.kv_rank + a.rot;
+  const int64_t kv_stride = (int64_t)a.heads * (dim + vdim);
+  const float4 zero = make_float4(0, 0, 0, 0);
+
+  for (int i = tid; i < AQ * (KP / 4); i += ROW_THREADS) {
+    const int r = i / (KP / 4), c = i % (KP / 4) * 4;
+    float4 v = zero;
+    if (t0 + r < t_count && c < hd)
+      v = *reinterpret_cast<const float4 *>(
+          q + ((int64_t)(t0 + r) * a.heads + head) * hd + c);
+    *reinterpret_cast<float4 *>(&sq[r][c]) = v;
+  }
+  float m[QN], l[QN];
+  float2 o[QN][CN][2];
+#pragma unroll
+  for (int i = 0; i < QN; ++i) {
+    m[i] = LOWEST;
+    l[i] = 0.0f;
+#pragma unroll
+    for (int c = 0; c < CN; ++c)
+      o[i][c][0] = o[i][c][1] = make_float2(0, 0);
+  }
+  const int first_key = max(0, base + t0 - a.window + 1);
+  const int last_key = base + min(t0 + AQ, t_count) - 1;
+  for (int k0 = first_key; k0 <= last_key; k0 += AK) {
+    const int row0 = k0 % a.cache_rows;
+    __syncthreads(); /* the tiles of the round before are done with */
+    for (int i = tid; i < AK * (KP / 4); i += ROW_THREADS) {
+      const int r = i / (KP / 4), c = i % (KP / 4) * 4;
+      float4 v = zero;
+      if (k0 + r <= last_key && c < hd) {
+        int row = row0 + r;
+        if (row >= a.cache_rows)
+          row -= a.cache_rows;
+        v = *reinterpret_cast<const float4 *>(
+            c < dim ? kv + (k0 + r - first) * kv_stride + head * (dim + vdim) + c
+                    : a.ring + (int64_t)row * row_floats + a.kv_rank + c - dim);
+      }
+      *reinterpret_cast<float4 *>(&sk[r][c]) = v;
+    }
+    for (int i = tid; i < AK * (VP / 4); i += ROW_THREADS) {
+      const int r = i / (VP / 4), c = i % (VP / 4) * 4;
+      float4 v = zero;
+      if (k0 + r <= last_key && c < vdim)
+        v = *reinterpret_cast<const float4 *>(kv + (k0 + r - first) * kv_stride +
+                                              head * (dim + vdim) + dim + c);
+      *reinterpret_cast<float4 *>(&sv[r][c]) = v;
+    }
+    __syncthreads();
+    float2 s2[QN][KN];
+#pragma unroll
+    for (int i = 0; i < QN; ++i)
+#pragma unroll
+      for (int j = 0; j < KN; ++j)
+        s2[i][j] = make_float2(0, 0);
+#pragma unroll 2
+    for (int d = 0; d < hd; d += 4) {
+      float4 qv[QN], kq[KN];
+#pragma unroll
+      for (int i = 0; i < QN; ++i)
+        qv[i] = *reinterpret_cast<const float4 *>(&sq[ty * QN + i][d]);
+#pragma unroll
+      for (int j = 0; j < KN; ++j)
+        kq[j] = *reinterpret_cast<const float4 *>(&sk[tx + 16 * j][d]);
+#pragma unroll
+      for (int i = 0; i < QN; ++i)
+#pragma unroll
+        for (int j = 0; j < KN; ++j) {
+          fma_pair(s2[i][j], make_float2(qv[i].x, qv[i].y), make_float2(kq[j].x, kq[j].y));
+          fma_pair(s2[i][j], make_float2(qv[i].z, qv[i].w), make_float2(kq[j].z, kq[j].w));
+        }
+    }
+#pragma unroll
+    for (int i = 0; i < QN; ++i) {
+      const int at = base + t0 + ty * QN + i;
+      bool seen[KN];
+      float s[KN], big = LOWEST;
+#pragma unroll
+      for (int j = 0; j < KN; ++j) {
+        const int behind = at - (k0 + tx + 16 * j);
+        seen[j] = behind >= 0 && behind < a.window;
+        s[j] = seen[j] ? (s2[i][j].x + s2[i][j].y) * a.scale : LOWEST;
+        big = fmaxf(big, s[j]);
+      }
+#pragma unroll
+      for (int off = 8; off > 0; off >>= 1)
+        big = fmaxf(big, __shfl_xor_sync(0xffffffffu, big, off));
+      const float mn = fmaxf(m[i], big);
+      const float fix = expf(m[i] - mn);
+      float sum = 0.0f;
+#pragma unroll
+      for (int j = 0; j < KN; ++j) {
+        const float w = seen[j] ? expf(s[j] - mn) : 0.0f;
+        sp[ty * QN + i][tx + 16 * j] = w;
+        sum += w;
+      }
+#pragma unroll
+      for (int off = 8; off > 0; off >>= 1)
+        sum += __shfl_xor_sync(0xffffffffu, sum, off);
+      l[i] = l[i] * fix + sum;
+      m[i] = mn;
+      const float2 fix2 = make_float2(fix, fix);
+#pragma unroll
+      for (int c = 0; c < CN; ++c) {
+        o[i][c][0] = mul_pair(o[i][c][0], fix2);
+        o[i][c][1] = mul_pair(o[i][c][1], fix2);
+      }
+    }
+    __syncwarp(); /* a query's weights stay within the half warp that made them */
+    for (int k = 0; k < AK; k += 4) {
+      float4 w[QN];
+#pragma unroll
+      for (int i = 0; i < QN; ++i)
+        w[i] = *reinterpret_cast<const float4 *>(&sp[ty * QN + i][k]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j)
+#pragma unroll
+        for (int c = 0; c < CN; ++c) {
+          const float4 v =
+              *reinterpret_cast<const float4 *>(&sv[k + j][tx * 4 + 64 * c]);
+#pragma unroll
+          for (int i = 0; i < QN; ++i) {
+            const float p = j == 0 ? w[i].x : j == 1 ? w[i].y : j == 2 ? w[i].z : w[i].w;
+            fma_pair(o[i][c][0], make_float2(p, p), make_float2(v.x, v.y));
+            fma_pair(o[i][c][1], make_float2(p, p), make_float2(v.z, v.w));
+          }
+        }
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < QN; ++i) {
+    const int t = t0 + ty * QN + i;
+    if (t >= t_count)
+      continue;
+#pragma unroll
+    for (int c = 0; c < CN; ++c) {
+      const int d = tx * 4 + 64 * c;
+      if (d >= vdim)
+        continue;
+      const float v[4] = {o[i][c][0].x / l[i], o[i][c][0].y / l[i], o[i][c][1].x / l[i],
+                          o[i][c][1].y / l[i]};
+      store_terms4(terms, cols, t, head * vdim + d, v);
+    }
+  }
+}
+
+const char *refuse(const LatentArgs &a) {
+  if (a.heads < 1 || (a.dim | a.rot | a.vdim) % 8 != 0 || a.dim < 8 || a.rot < 0 ||
+      a.vdim < 8 || a.dim + a.rot > 512 || a.vdim > 512 || a.kv_rank < 64 ||
+      a.kv_rank % 64 != 0 || a.kv_rank + a.rot > 1024)
+    return "latent attention takes head sizes in multiples of 8 and a latent in "
+           "multiples of 64; keys and values of at most 512, latent and rotated part "
+           "of at most 1024 values";
+  if (a.window < 1 || a.cache_rows < 1)
+    return "a window holds at least its own token";
+  if (((uintptr_t)a.ring | (uintptr_t)a.w_ukv | (uintptr_t)a.w_uk_t) & 15 ||
+      a.ring_batch_stride % 4 != 0)
+    return "the ring and the matrices of latent attention must be 16-byte aligned";
+  return nullptr;
+}
+
+struct StepCall {
+  const float *q;
+  int64_t q_stride;
+  const float *down;
+  int64_t down_stride;
+  int batch;
+  float *out;
+  int64_t out_stride;
+  cudaStream_t stream;
+};
+
+template <typename W, int GH, int D4>
+const char *launch_step(const LatentArgs &a, const StepCall &c) {
+  constexpr int NW = 8;
+  const int smem = latent_smem(GH, D4, NW, a.dim, a.kv_rank) * (int)sizeof(float);
+  constexpr int most = latent_smem(GH, D4, NW, 512, D4 * 128) * (int)sizeof(float);
+  static_assert(most <= 200 * 1024, "the arrays fit in shared memory");
+  if (allow_dynamic_smem((const void *)latent_decode_kernel<W, GH, D4, NW>, most) !=
+      cudaSuccess)
+    return "latent attention could not get its shared memory";
+  launch_chained_cluster_smem(latent_decode_kernel<W, GH, D4, NW>,
+                              dim3(CL, (a.heads + GH - 1) / GH, c.batch), dim3(NW * 32),
+                              CL, smem, c.stream, a, c.q, c.q_stride, c.down,
+                              c.down_stride, c.out, c.out_stride);
+  return check_launch("a step of latent attention");
+}
+
+template <typename W, int D4>
+const char *launch_step_heads(const LatentArgs &a, const StepCall &c) {
+  /* as many heads a cluster as keep the grid within one wave */
+  const int64_t clusters = (int64_t)a.heads * c.batch;
+  if (clusters * CL <= sm_count())
+    return launch_step<W, 1, D4>(a, c);
+  if (D4 > 2 || clusters * CL <= 2 * sm_count())
+    return launch_step<W, 2, D4>(a, c);
+  return launch_step<W, (D4 > 2 ? 2 : 4), D4>(a, c);
+}
+
+template <typename W> const char *launch_step_row(const LatentArgs &a, const StepCall &c) {
+  const int row = a.kv_rank + a.rot;
+  if (row <= 128)
+    return launch_step_heads<W, 1>(a, c);
+  if (row <= 256)
+    return launch_step_heads<W, 2>(a, c);
+  if (row <= 640)
+    return launch_step_heads<W, 5>(a, c);
+  return launch_step_heads<W, 8>(a, c);
+}
+
+template <int KP, int VP, int AQ, int AK>
+const char *launch_rows(const LatentArgs &a, const float *q, const float *kv, int first,
+                        int t, __nv_bfloat16 *terms, int cols, cudaStream_t stream) {
+  constexpr int smem = rows_smem(KP, VP, AQ, AK);
+  if (allow_dynamic_smem((const void *)latent_rows_kernel<KP, VP, AQ, AK>, smem) !=
+      cudaSuccess)
+    return "the multi-position latent attention could not get its shared memory";
+  launch_chained(latent_rows_kernel<KP, VP, AQ, AK>, dim3((t + AQ - 1) / AQ, a.heads),
+                 dim3(ROW_THREADS), smem, stream, a, q, kv, first, t, terms, cols);
+  return check_launch("the multi-position latent attention");
+}
+
+} // namespace
+
+const char *latent_attention_decode(const LatentArgs &a, const float *q, int64_t q_stride,
+                                    const float *down, int64_t down_stride, int batch,
+                                    float *out, int64_t out_stride, cudaStream_t stream) {
+  if (const char *why = refuse(a))
+    return why;
+  if (a.cache_rows < a.window)
+    return "the ring must hold a window";
+  if ((((uintptr_t)q | (uintptr_t)down) & 7) || (q_stride | down_stride) % 2 != 0)
+    return "queries and latents must be 8-byte aligned";
+  const StepCall c{q, q_stride, down, down_stride, batch, out, out_stride, stream};
+  return a.fmt == kFmtBf16 ? launch_step_row<__nv_bfloat16>(a, c)
+                           : launch_step_row<float>(a, c);
+}
+
+const char *latent_rows_down(const LatentArgs &a, const float *partials, int splits, int t,
+                             int q_rank, const float *q_gain, int q_mean, void *terms,
+                             cudaStream_t stream) {
+  if (const char *why = refuse(a))
+    return why;
+  const int smem = (q_rank + a.kv_rank) * (int)sizeof(float);
+  if (smem > 200 * 1024 ||
+      allow_dynamic_smem((const void *)latent_down_kernel, 200 * 1024) != cudaSuccess)
+    return "the two latents of a position must fit in shared memory";
+  launch_chained(latent_down_kernel, dim3(t), dim3(256), smem, stream, a, partials, splits,
+                 t, q_rank, q_gain, q_mean, (__nv_bfloat16 *)terms);
+  return check_launch("the latents of a prompt");
+}
+
+const char *latent_rows_q(const LatentArgs &a, const float *partials, int splits, int t,
+                          float *q, cudaStream_t stream) {
+  if (const char *why = refuse(a))
+    return why;
+  const int64_t count = (int64_t)t * (a.heads * (a.dim + a.rot) / 4);
+  launch_chained(latent_q_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0,
+                 stream, a, partials, splits, t, q);
+  return check_launch("the queries of a prompt");
+}
+
+const char *latent_rows_gather(const LatentArgs &a, int first, int n, void *terms,
+                               cudaStream_t stream) {
+  if (const char *why = refuse(a))
+    return why;
+  const int64_t count = (int64_t)n * (a.kv_rank / 8);
+  launch_chained(latent_gather_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0,
+                 stream, a, first, n, (__nv_bfloat16 *)terms);
+  return check_launch("the latents of a window");
+}
+
+const char *latent_attention_rows(const LatentArgs &a, const float *q, const float *kv,
+                                  int first, int t, void *terms, int cols,
+                                  cudaStream_t stream) {
+  if (const char *why = refuse(a))
+    return why;
+  if (cols % 4 != 0 || cols < a.heads * a.vdim)
+    return "the output has too few columns";
+  __nv_bfloat16 *to = (__nv_bfloat16 *)terms;
+  const int hd = a.dim + a.rot;
+  if (hd <= 64 && a.vdim <= 64)
+    return launch_rows<64, 64, 64, 64>(a, q, kv, first, t, to, cols, stream);
+  if (hd <= 128 && a.vdim <= 128)
+    return launch_rows<128, 128, 64, 32>(a, q, kv, first, t, to, cols, stream);
+  if (hd <= 192 && a.vdim <= 128)
+    return launch_rows<192, 128, 64, 32>(a, q, kv, first, t, to, cols, stream);
+  if (hd <= 256 && a.vdim <= 256)
+    return launch_rows<256, 256, 64, 32>(a, q, kv, first, t, to, cols, stream);
+  return launch_rows<512, 512, 32, 32>(a, q, kv, first, t, to, cols, stream);
+}
+
+} // namespace vxb

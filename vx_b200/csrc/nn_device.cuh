@@ -46,6 +46,51 @@ __device__ __forceinline__ float squared_relu(float v) {
   return r * r;
 }
 
+/* z times the normal distribution function of z, without the cancellation that
+   1 + erf(z / sqrt 2) has far below zero */
+__device__ __forceinline__ float gelu(float z) {
+  return 0.5f * z * erfcf(-0.70710678118654752f * z);
+}
+__device__ __forceinline__ float silu(float z) { return z * sigmoid(z); }
+/* cap * tanh(scale * v / cap); cap 0: scale * v */
+__device__ __forceinline__ float capped_logit(float v, float scale, float cap) {
+  v *= scale;
+  return cap > 0.0f ? cap * tanhf(v / cap) : v;
+}
+
+/* Sine and cosine at a position whose angle advances by `turns` of a full turn per
+   position: what is left of the angle after whole turns is exact enough in f64 for
+   any position, and small in f32. */
+__device__ __forceinline__ void turned(int pos, double turns, float &sine,
+                                       float &cosine) {
+  const double t = pos * turns;
+  sincospif(2.0f * (float)(t - rint(t)), &sine, &cosine);
+}
+
+/* d += a * b, and a * b, on two values at once (one instruction on sm_100) */
+__device__ __forceinline__ void fma_pair(float2 &d, const float2 a, const float2 b) {
+  unsigned long long dd = *reinterpret_cast<unsigned long long *>(&d);
+  asm("fma.rn.f32x2 %0, %1, %2, %0;"
+      : "+l"(dd)
+      : "l"(*reinterpret_cast<const unsigned long long *>(&a)),
+        "l"(*reinterpret_cast<const unsigned long long *>(&b)));
+  d = *reinterpret_cast<float2 *>(&dd);
+}
+__device__ __forceinline__ float2 mul_pair(const float2 a, const float2 b) {
+  unsigned long long dd;
+  asm("mul.rn.f32x2 %0, %1, %2;"
+      : "=l"(dd)
+      : "l"(*reinterpret_cast<const unsigned long long *>(&a)),
+        "l"(*reinterpret_cast<const unsigned long long *>(&b)));
+  return *reinterpret_cast<float2 *>(&dd);
+}
+__device__ __forceinline__ void axpy(float4 &y, float a, const float4 &x) {
+  y.x = fmaf(a, x.x, y.x);
+  y.y = fmaf(a, x.y, y.y);
+  y.z = fmaf(a, x.z, y.z);
+  y.w = fmaf(a, x.w, y.w);
+}
+
 /* The pushed exchange moves (value, call) pairs: an aligned 8-byte store
    arrives whole, so a pair that carries the expected call number is complete
    and is its own arrival flag. An item's two rows travel as two pairs in one
@@ -389,7 +434,13 @@ attention_unit(const AttnArgs &a, int split_idx, int y, int b, int warp,
  * rows whose results the epilogue needs together; a warp owns a contiguous,
  * balanced range of items and streams both rows of an item at once. */
 enum { EPI_STORE = 0, EPI_ADD = 1, EPI_BIAS = 2, EPI_SWIGLU = 3, EPI_QKV = 4,
-       EPI_PUSH = 5, EPI_FAN = 6 };
+       EPI_PUSH = 5, EPI_FAN = 6,
+       /* a residual of several streams (stream_proj in kernels.h): in front the
+          weighted sum of the streams and its norm, or behind the streams' mixing */
+       EPI_IN_STORE = 7, EPI_IN_GELU = 8, EPI_IN_LOGITS = 9, EPI_MIX = 10 };
+__host__ __device__ constexpr bool reads_streams(int epi) {
+  return epi == EPI_IN_STORE || epi == EPI_IN_GELU || epi == EPI_IN_LOGITS;
+}
 
 struct RowDotParams {
   /* weights */
@@ -438,6 +489,11 @@ struct RowDotParams {
   int norm_n;
   /* EPI_FAN (see FanOut in kernels.h) */
   FanOut fan;
+  /* EPI_IN_*, EPI_MIX (see StreamProj in kernels.h) */
+  int streams;
+  int64_t stream_stride;
+  const float *stream_in, *stream_mix, *stream_out;
+  float logit_scale, logit_cap;
 };
 
 /* The projection kernel by weight format (rowdot_f32.cu, rowdot_bf16.cu,
@@ -448,7 +504,11 @@ const char *rowdot_quant(int epi, RowDotParams &p, int fmt, cudaStream_t stream)
 int rowdot_f32_status();
 int rowdot_bf16_status();
 int rowdot_quant_status();
-
+/* EPI_IN_*, EPI_MIX: rowdot_streams_f32.cu, rowdot_streams_bf16.cu */
+const char *rowdot_streams_f32(int epi, RowDotParams &p, cudaStream_t stream);
+const char *rowdot_streams_bf16(int epi, RowDotParams &p, cudaStream_t stream);
+int rowdot_streams_f32_status();
+int rowdot_streams_bf16_status();
 
 namespace {
 

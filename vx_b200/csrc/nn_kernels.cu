@@ -71,6 +71,9 @@ const char *launch_rowdot(int epi, RowDotParams &p, int fmt, cudaStream_t stream
       return "the quantised projections are not sharded";
     return rowdot_quant(epi, p, fmt, stream);
   }
+  if (reads_streams(epi) || epi == EPI_MIX)
+    return fmt == kFmtBf16 ? rowdot_streams_bf16(epi, p, stream)
+                           : rowdot_streams_f32(epi, p, stream);
   return fmt == kFmtBf16 ? rowdot_bf16(epi, p, stream) : rowdot_f32(epi, p, stream);
 }
 
@@ -365,6 +368,44 @@ const char *fan_proj(const FanArgs &a, cudaStream_t stream) {
   return launch_rowdot(EPI_FAN, p, a.fmt, stream);
 }
 
+const char *stream_proj(const StreamProj &a, cudaStream_t stream) {
+  if (a.streams < 1 || a.streams > kMaxStreams)
+    return "a residual has 1 to 32 streams";
+  if (a.rows % 2 != 0 || a.y_stride % 2 != 0 || a.stream_stride % 4 != 0)
+    return "the projections around streams take an even number of rows, and streams "
+           "a multiple of 4 values apart";
+  RowDotParams p{};
+  p.w0 = a.w;
+  p.rows = a.rows;
+  p.cols = a.cols;
+  p.items = a.rows / 2;
+  p.x = a.x;
+  p.x_stride = a.x_stride;
+  p.batch = a.batch;
+  p.norm_w = a.norm_w;
+  p.norm_n = a.norm_n;
+  p.eps = a.eps;
+  p.y = a.y;
+  p.y_stride = a.y_stride;
+  p.streams = a.streams;
+  p.stream_stride = a.stream_stride;
+  p.stream_in = a.in;
+  p.stream_mix = a.mix;
+  p.stream_out = a.out;
+  p.logit_scale = a.logit_scale;
+  p.logit_cap = a.logit_cap;
+  switch (a.mode) {
+  case kStreamsStore: return launch_rowdot(EPI_IN_STORE, p, a.fmt, stream);
+  case kStreamsGelu: return launch_rowdot(EPI_IN_GELU, p, a.fmt, stream);
+  case kStreamsLogits: return launch_rowdot(EPI_IN_LOGITS, p, a.fmt, stream);
+  case kStreamsMix:
+    if (!a.mix || !a.out)
+      return "mixing streams takes their matrix and the weights of the product";
+    return launch_rowdot(EPI_MIX, p, a.fmt, stream);
+  default: return "unknown mode of a projection around streams";
+  }
+}
+
 const char *swiglu(const SwigluArgs &a, cudaStream_t stream) {
   if (a.rows <= 0 || a.batch <= 0)
     return nullptr;
@@ -444,7 +485,8 @@ int tp_status(cudaStream_t stream) {
   if (cudaStreamSynchronize(stream) != cudaSuccess)
     return -1;
   const int b = rowdot_bf16_status(), f = rowdot_f32_status(), q = rowdot_quant_status();
-  return b ? b : (f ? f : q);
+  const int sb = rowdot_streams_bf16_status(), sf = rowdot_streams_f32_status();
+  return b ? b : f ? f : q ? q : sb ? sb : sf;
 }
 
 const char *rms_norm(float *y, const float *x, const void *w, bool wbf16, int n,

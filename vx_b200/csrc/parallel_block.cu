@@ -29,10 +29,12 @@ __global__ void __launch_bounds__(1024) position_embed_kernel(const PositionEmbe
   const int64_t t = blockIdx.x;
   const int token = a.tokens[t];
   const int pos = a.per_sequence ? a.positions[t] : a.positions[0] + (int)t;
-  float *row = a.x + t * a.dim;
+  const int copies = a.copies > 1 ? a.copies : 1;
+  float *row = a.x + t * copies * a.dim;
   if (token < 0 || token >= a.vocab) {
     for (int i = threadIdx.x; i < a.dim; i += blockDim.x)
-      row[i] = i < a.width ? __int_as_float(0x7fc00000) : 0.0f;
+      for (int c = 0; c < copies; ++c)
+        row[c * a.dim + i] = i < a.width ? __int_as_float(0x7fc00000) : 0.0f;
     return;
   }
   float ss = 0.0f;
@@ -48,11 +50,9 @@ __global__ void __launch_bounds__(1024) position_embed_kernel(const PositionEmbe
     } else {
       e = ((const float2 *)a.table)[((int64_t)token * a.dim >> 1) + k];
     }
-    /* the angle in turns: what is left of it after whole turns is exact enough
-       in f64 for any position, and small in f32 */
-    const double turns = pos * a.turns[k];
-    float sine, cosine;
-    sincospif(2.0f * (float)(turns - rint(turns)), &sine, &cosine);
+    float sine = 0.0f, cosine = 0.0f;
+    if (a.turns)
+      turned(pos, a.turns[k], sine, cosine);
     const float v0 = fmaf(e.x, a.scale, sine);
     const float v1 = 2 * k + 1 < a.width ? fmaf(e.y, a.scale, cosine) : 0.0f;
     *reinterpret_cast<float2 *>(&embed_row[2 * k]) = make_float2(v0, v1);
@@ -67,8 +67,13 @@ __global__ void __launch_bounds__(1024) position_embed_kernel(const PositionEmbe
   for (int k = 0; k < (int)blockDim.x / 32; ++k) /* fixed order */
     total += red[k];
   const float inv = 1.0f / sqrtf(total / (float)a.width + a.eps);
-  for (int i = threadIdx.x; i < a.dim; i += blockDim.x)
-    row[i] = i < a.width ? embed_row[i] * inv * a.gain[i] : 0.0f;
+  for (int i = threadIdx.x; i < a.dim; i += blockDim.x) {
+    const float v = i >= a.width ? 0.0f
+                    : a.gain     ? embed_row[i] * inv * a.gain[i]
+                                 : embed_row[i];
+    for (int c = 0; c < copies; ++c)
+      row[c * a.dim + i] = v;
+  }
 }
 
 /* ---- after the input GEMM: a thread per (position, eight rows) ---------------- */
@@ -111,14 +116,16 @@ fan_finish_kernel(const float *partials, int splits, int t_count, int n,
 }
 
 __global__ void __launch_bounds__(256)
-sum_kernel(float *out, const float *partials, int splits, int t_count, int n) {
+sum_kernel(float *out, const float *partials, int splits, int t_count, int n, float scale,
+           float cap) {
   chain_release();
   chain_wait();
   const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= (int64_t)t_count * n)
     return;
   const int64_t t = idx / n;
-  out[idx] = sum_runs(partials, splits, t_count, n, t, idx - t * n);
+  out[idx] = capped_logit(sum_runs(partials, splits, t_count, n, t, idx - t * n), scale,
+                          cap);
 }
 
 /* ---- the f32 product on the FP32 pipe: 64 positions x 64 rows a block, 4 x 4 a
@@ -209,10 +216,10 @@ const char *rows_fan_finish(const float *partials, int splits, int t, int n,
 }
 
 const char *rows_sum(float *out, const float *partials, int splits, int t, int n,
-                     cudaStream_t stream) {
+                     cudaStream_t stream, float scale, float cap) {
   const int64_t count = (int64_t)t * n;
   launch_chained(sum_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0, stream,
-                 out, partials, splits, t, n);
+                 out, partials, splits, t, n, scale, cap);
   return check_launch("the sum of a product's runs");
 }
 

@@ -53,15 +53,6 @@ __device__ __forceinline__ void unpack_fp8(const uint4 &wv, float (&wf)[16]) {
     }
   }
 }
-/* d += a * b on two values at once (one instruction on sm_100) */
-__device__ __forceinline__ void fma_pair(float2 &d, const float2 a, const float2 b) {
-  unsigned long long dd = *reinterpret_cast<unsigned long long *>(&d);
-  asm("fma.rn.f32x2 %0, %1, %2, %0;"
-      : "+l"(dd)
-      : "l"(*reinterpret_cast<const unsigned long long *>(&a)),
-        "l"(*reinterpret_cast<const unsigned long long *>(&b)));
-  d = *reinterpret_cast<float2 *>(&dd);
-}
 __device__ __forceinline__ float2 add_pair(const float2 a, const float2 b) {
   unsigned long long dd;
   asm("add.rn.f32x2 %0, %1, %2;"
@@ -350,7 +341,14 @@ rowdot_kernel(const RowDotParams p) {
           const int q = q0 + k * blockDim.x;
           v[k] = wn[k] = make_float4(0, 0, 0, 0);
           if (q < quads) {
-            v[k] = px4[q];
+            if constexpr (reads_streams(EPI)) {
+              /* the weighted sum of the streams takes the place of x */
+              for (int s = 0; s < p.streams; ++s)
+                axpy(v[k], p.stream_in ? p.stream_in[s] : 1.0f,
+                     px4[s * (p.stream_stride / 4) + q]);
+            } else {
+              v[k] = px4[q];
+            }
             if (p.norm_bf16) {
               const uint2 w = reinterpret_cast<const uint2 *>(p.norm_w)[q];
               wn[k] = make_float4(bf_lo(w.x), bf_hi(w.x), bf_lo(w.y), bf_hi(w.y));
@@ -489,6 +487,12 @@ rowdot_kernel(const RowDotParams p) {
         }
       }
     }
+    if (early && EPI == EPI_MIX && ch == 0 && lane < p.streams) {
+      const float2 old =
+          *reinterpret_cast<const float2 *>(p.y + lane * p.stream_stride + 2 * item);
+      pre0 = old.x;
+      pre1 = old.y;
+    }
     if (++next_ch == nch) {
       next_ch = 0;
       ++next_item;
@@ -590,13 +594,39 @@ rowdot_kernel(const RowDotParams p) {
       }
       continue;
     }
+    if constexpr (EPI == EPI_MIX) {
+      /* Lane t makes stream t of the item's two rows, from all the old streams
+         (lane s holds stream s's) and the product, which every lane has. */
+      const int streams = p.streams;
+#pragma unroll
+      for (int b = 0; b < B; ++b) {
+        float *at = p.y + b * p.y_stride + lane * p.stream_stride + 2 * item;
+        float2 old = make_float2(pre0, pre1);
+        if (!early)
+          old = lane < streams ? *reinterpret_cast<const float2 *>(at)
+                               : make_float2(0, 0);
+        float2 now = make_float2(0, 0);
+        if (lane < streams) {
+          const float out = p.stream_out[lane];
+          now = make_float2(out * t0[b], out * t1[b]);
+        }
+        for (int s = 0; s < streams; ++s) {
+          const float m = lane < streams ? p.stream_mix[s * streams + lane] : 0.0f;
+          now.x = fmaf(m, __shfl_sync(0xffffffffu, old.x, s), now.x);
+          now.y = fmaf(m, __shfl_sync(0xffffffffu, old.y, s), now.y);
+        }
+        if (lane < streams)
+          *reinterpret_cast<float2 *>(at) = now;
+      }
+      continue;
+    }
     if (lane != 0)
       continue;
 
     /* ---- epilogue, lane 0 ---- */
 #pragma unroll
     for (int b = 0; b < B; ++b) {
-      if (EPI == EPI_STORE || EPI == EPI_ADD || EPI == EPI_BIAS) {
+      if (EPI == EPI_STORE || EPI == EPI_ADD || EPI == EPI_BIAS || reads_streams(EPI)) {
         float *y = p.y + b * p.y_stride;
         const int ra = 2 * item, rb = 2 * item + 1;
         float v0 = t0[b], v1 = t1[b];
@@ -612,6 +642,12 @@ rowdot_kernel(const RowDotParams p) {
           v0 += bf16_at(p.bias, ra);
           if (r1)
             v1 += bf16_at(p.bias, rb);
+        } else if (EPI == EPI_IN_GELU) {
+          v0 = gelu(v0);
+          v1 = gelu(v1);
+        } else if (EPI == EPI_IN_LOGITS) {
+          v0 = capped_logit(v0, p.logit_scale, p.logit_cap);
+          v1 = capped_logit(v1, p.logit_scale, p.logit_cap);
         }
         y[ra] = v0;
         if (r1)

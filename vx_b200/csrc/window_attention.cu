@@ -38,13 +38,6 @@ template <int GH, int D4, int NW> struct WindowShared {
   __align__(16) float acc[NW][GH][D4 * 128];
 };
 
-__device__ __forceinline__ void axpy(float4 &y, float a, const float4 &x) {
-  y.x = fmaf(a, x.x, y.x);
-  y.y = fmaf(a, x.y, y.y);
-  y.z = fmaf(a, x.z, y.z);
-  y.w = fmaf(a, x.w, y.w);
-}
-
 template <int GH, int D4, int NW>
 __global__ void __launch_bounds__(NW * 32)
 window_decode_kernel(const WindowAttnArgs a, float *out, int64_t out_stride) {

@@ -149,7 +149,7 @@ def decoder_of(config, tensors, bf16, max_seq, batch=1, prefill_rows=0, keep=Non
         eps=config.eps, embed_scale=config.embed_scale, embed=tensors["embed"],
         classifier=tensors["embed"], embed_norm=tensors["embed_norm"],
         final_norm=tensors["final_norm"], turns=tensors["turns"], layers=layers)
-    return Decoder.from_parallel(cfg, keep=(keep, layers))
+    return Decoder.from_config(cfg, keep=(keep, layers))
 
 
 def from_tensors(config, tensor, dtype="bfloat16", max_seq=4096, batch=1,

@@ -47,7 +47,7 @@ EXTRA_SYMBOLS = [
     "vx_decoder_create", "vx_decoder_destroy", "vx_decoder_reset",
     "vx_decoder_step", "vx_decoder_prefill", "vx_decoder_logits",
     "vx_decoder_logits_pitch", "vx_decoder_create_parallel",
-    "vx_decoder_prefill_logits",
+    "vx_decoder_create_streams", "vx_decoder_prefill_logits",
     "vx_decoder_kernels_per_step",
     "vx_decoder_step_trace",
     "vx_decoder_kv_cache", "vx_decoder_kv_cache_bytes", "vx_decoder_adopt_kv",
@@ -98,6 +98,35 @@ class ParallelConfig(C.Structure):
                [(n, C.c_void_p) for n in
                 ("embed", "classifier", "embed_norm", "final_norm", "turns")] + \
                [("layers", C.POINTER(ParallelLayer))]
+
+
+class StreamMix(C.Structure):
+    _fields_ = [(n, C.c_void_p) for n in ("hc_in", "mix", "out")]
+
+
+class StreamLayer(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in
+                ("kind", "heads", "dim", "vdim", "rot_dim", "q_rank", "q_mean",
+                 "kv_rank", "kv_mean", "window", "a_rank", "v_mean", "hidden")] + \
+               [(n, C.c_float) for n in ("scale", "inv_tau")] + \
+               [(n, C.c_void_p) for n in
+                ("norm1", "w_in", "w_o", "q_norm", "kv_norm", "w_uq", "w_ukv",
+                 "w_uk_t", "turns", "a2", "a2_bias", "o_norm", "norm2", "w_up",
+                 "w_down")] + \
+               [("hc1", StreamMix), ("hc2", StreamMix)]
+
+
+class StreamConfig(C.Structure):
+    _fields_ = [(n, C.c_int32) for n in
+                ("width", "dim", "n_layers", "vocab", "vocab_rows", "max_seq",
+                 "weights_bf16", "batch", "prefill_rows", "streams")] + \
+               [(n, C.c_float) for n in
+                ("eps", "embed_scale", "logit_scale", "logit_cap")] + \
+               [(n, C.c_void_p) for n in ("embed", "classifier", "final_norm")] + \
+               [("layers", C.POINTER(StreamLayer))]
+
+
+MIXER_LATENT, MIXER_GATED_LINEAR = 1, 2
 
 
 class Llama2cConfig(C.Structure):
@@ -169,6 +198,8 @@ def lib():
     L.vx_decoder_prefill.argtypes = [vp, vp, i32]
     L.vx_decoder_create_parallel.restype = vp
     L.vx_decoder_create_parallel.argtypes = [C.POINTER(ParallelConfig)]
+    L.vx_decoder_create_streams.restype = vp
+    L.vx_decoder_create_streams.argtypes = [C.POINTER(StreamConfig)]
     L.vx_decoder_prefill_logits.restype = i32
     L.vx_decoder_prefill_logits.argtypes = [vp, vp, i32, vp, i32, vp]
     L.vx_decoder_logits_pitch.restype = i32

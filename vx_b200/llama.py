@@ -14,7 +14,8 @@ import ctypes as C
 import numpy as np
 
 from . import abi
-from .lib import DecoderConfig, DecoderWeights, Llama2cConfig, ParallelConfig, lib
+from .lib import (DecoderConfig, DecoderWeights, Llama2cConfig, ParallelConfig,
+                  StreamConfig, lib)
 
 
 def _ptr_array(ptrs):
@@ -51,10 +52,12 @@ class Decoder:
         return self
 
     @classmethod
-    def from_parallel(cls, cfg, keep=None):
-        """A decoder of parallel blocks (vx_decoder_create_parallel); cfg is a
-        ParallelConfig, `keep` holds whatever owns its memory."""
-        handle = lib().vx_decoder_create_parallel(C.byref(cfg))
+    def from_config(cls, cfg, keep=None):
+        """A decoder of parallel blocks (cfg a ParallelConfig) or of several residual
+        streams (a StreamConfig); `keep` holds whatever owns its memory."""
+        create = lib().vx_decoder_create_parallel if isinstance(cfg, ParallelConfig) \
+            else lib().vx_decoder_create_streams
+        handle = create(C.byref(cfg))
         if not handle:
             raise ValueError(lib().vx_b200_last_error().decode())
         self = cls.__new__(cls)
@@ -118,7 +121,7 @@ class Decoder:
         in one pass where the decoder has one that gives logits, single steps
         otherwise."""
         tokens, want = [int(t) for t in tokens], [int(w) for w in want]
-        if isinstance(self.cfg, ParallelConfig) and len(tokens) > 1:
+        if isinstance(self.cfg, (ParallelConfig, StreamConfig)) and len(tokens) > 1:
             arr = (C.c_int32 * len(tokens))(*tokens)
             places = (C.c_int32 * max(len(want), 1))(*want)
             out = np.empty((len(want), self.cfg.vocab), np.float32)

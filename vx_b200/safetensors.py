@@ -31,10 +31,16 @@ class SafeTensors:
     def names(self):
         return list(self._entries)
 
-    def _array(self, name):
+    def _entry(self, name):
         if name not in self._entries:
             raise ValueError("%s has no tensor %r" % (self._path, name))
-        e = self._entries[name]
+        return self._entries[name]
+
+    def shape(self, name):
+        return tuple(self._entry(name)["shape"])
+
+    def _array(self, name):
+        e = self._entry(name)
         if e["dtype"] not in _NUMPY:
             raise ValueError("tensor %r has the type %s" % (name, e["dtype"]))
         lo, hi = e["data_offsets"]

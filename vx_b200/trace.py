@@ -56,6 +56,8 @@ def main(argv=None):
     args = ap.parse_args(argv)
 
     from . import models
+    from .lib import use
+    use(models.library(args.model))
     try:
         decoder = models.load(args.model, args.dtype, max(args.max_tokens, 1))
     except models.UnsupportedDtype as e:
