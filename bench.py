@@ -11,7 +11,7 @@ sequences per step), each with its error against the CPU oracle on sampled
 rows, the roofline of the dominant kernel, and the CPU baseline.
 
   python bench.py [--gpus N] [--steps K] [--warmup W] [--impl reference]
-  python bench.py --design gofilorn      another design beside the Llama decoder
+  python bench.py --design vamalix       another design beside the closest decoder
 """
 import argparse
 import ctypes as C
@@ -916,9 +916,11 @@ def run_ours(args):
         dist.destroy_process_group()
 
 
-# ---- another design beside the Llama decoder of equal size -------------------------
-# Layers like a real model's, in two widths; the Llama decoder beside each has the
-# same width, heads and number of weights a layer within 1 % (one key head as well).
+# ---- another design beside the closest decoder of equal size ------------------------
+# Layers like a real model's, in two widths. Beside Gofilorn stands a Llama decoder of
+# the same width, heads and number of weights a layer within 1 % (one key head as well);
+# beside Vamalix, whose two kinds of layer alternate, a Gofilorn decoder of the same
+# width, heads, window, number of layers and weights in all within 1 %.
 DESIGN_SIZES = {
     "width2048": dict(width=2048, heads=16, ff=7424, window=1024, layers=16,
                       llama_hidden=5632),
@@ -928,10 +930,10 @@ DESIGN_SIZES = {
 DESIGN_VOCAB, DESIGN_PROMPTS = 32000, (512, 2048)
 
 
-def gofilorn_of_size(s):
+def gofilorn_of_size(s, ff=None):
     """(decoder, bytes of weights a step streams) of random weights."""
     from vx_b200 import gofilorn
-    entry = dict(type="attention", mlp=dict(kind="dense", ff=s["ff"]),
+    entry = dict(type="attention", mlp=dict(kind="dense", ff=ff or s["ff"]),
                  mixer=dict(heads=s["heads"], kv_heads=1, dim=128, vdim=128,
                             mask=dict(size=s["window"]), scale=128 ** -0.5))
     cfg = gofilorn.GofilornConfig.from_dict(dict(
@@ -941,12 +943,56 @@ def gofilorn_of_size(s):
     return gofilorn.synthetic(cfg, MAX_SEQ), 2 * (weights + DESIGN_VOCAB * cfg.dim)
 
 
+def vamalix_config(s):
+    """(configuration, weights of its layers)"""
+    from vx_b200 import vamalix
+    latent = dict(type="latent_attention", mlp=dict(kind="dense", ff=s["ff"]),
+                  mixer=dict(heads=s["heads"], dim=128, rot_dim=64, vdim=128,
+                             kv_rank=512, q_rank=1536, scale=192 ** -0.5,
+                             rot=dict(base=10000.0, dims=64),
+                             mask=dict(size=s["window"])))
+    linear = dict(type="gla", mlp=None,
+                  mixer=dict(heads=s["width"] // 512, dim=256, vdim=512, tau=16.0))
+    cfg = vamalix.VamalixConfig.from_dict(dict(
+        architecture="Vamalix", width=s["width"], vocab=DESIGN_VOCAB, streams=4,
+        embedding=dict(scale=1.0), norm=dict(eps=1e-5), logit_scale=1.0,
+        logit_softcap=30.0, loop=None, layers=[latent, linear] * (s["layers"] // 2)))
+    weights = 0
+    for l in cfg.layers:
+        if l.kind == vamalix.MIXER_GATED_LINEAR:
+            l.set_rank(16)
+        weights += (l.in_rows + l.out_cols + 2 * l.hidden) * cfg.dim + sum(
+            rows * cols for rows, cols in l.inner)
+    return cfg, weights
+
+
+def vamalix_of_size(s):
+    from vx_b200 import vamalix
+    cfg, weights = vamalix_config(s)
+    return vamalix.synthetic(cfg, MAX_SEQ), 2 * (weights + DESIGN_VOCAB * cfg.dim)
+
+
+def gofilorn_like_vamalix(s):
+    cfg, weights = vamalix_config(s)
+    att = s["heads"] * 128
+    per_layer = weights / s["layers"] / s["width"]        # rows and columns of a layer
+    ff = round((per_layer - 3 * att - 128) / 2 / 64) * 64
+    return gofilorn_of_size(s, ff)
+
+
 def llama_of_size(s):
     from vx_b200 import llama
     shape = dict(dim=s["width"], hidden=s["llama_hidden"], n_layers=s["layers"],
                  q_heads=s["heads"], kv_heads=1, head_dim=128, vocab=DESIGN_VOCAB)
     return (llama.nn_bf16_model(max_seq=MAX_SEQ, **shape)[0],
             llama.weight_bytes_per_token(**shape))
+
+
+# design -> itself and the decoder beside it
+DESIGNS = {
+    "gofilorn": (("gofilorn", gofilorn_of_size), ("llama", llama_of_size)),
+    "vamalix": (("vamalix", vamalix_of_size), ("gofilorn", gofilorn_like_vamalix)),
+}
 
 
 def time_decoder(torch, dec, peaks, weight_bytes, steps, warmup):
@@ -985,8 +1031,8 @@ def time_decoder(torch, dec, peaks, weight_bytes, steps, warmup):
 
 
 def run_design(args):
-    """--design gofilorn: prefill and decode of the design at a few sizes, random
-    weights, one sequence, with the Llama decoder of equal size beside it."""
+    """--design: prefill and decode of the design at a few sizes, random weights, one
+    sequence, with the closest decoder of equal size beside it."""
     import torch
     from vx_b200 import ops
     peaks = measured_peaks()
@@ -996,7 +1042,7 @@ def run_design(args):
             if args.design_size and name != args.design_size:
                 continue
             row = dict(size=s)
-            for which, make in (("gofilorn", gofilorn_of_size), ("llama", llama_of_size)):
+            for which, make in DESIGNS[args.design]:
                 if args.design_only and which != args.design_only:
                     continue
                 dec, weight_bytes = make(s)
@@ -1008,7 +1054,7 @@ def run_design(args):
                 torch.cuda.empty_cache()
             sizes[name] = row
     print(json.dumps(dict(
-        metric="gofilorn_beside_llama", unit="tokens/s", steps=args.steps,
+        metric="_beside_".join(which for which, _ in DESIGNS[args.design]), unit="tokens/s", steps=args.steps,
         warmup=args.warmup, dtype="bf16 weights, f32 activations and accumulate",
         data="synthetic", higher_is_better=True, sizes=sizes,
         kernel_status=ops.kernel_status(), peaks=peaks, clocks=clocks.summary(),
@@ -1023,12 +1069,12 @@ def main():
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--no-extras", action="store_true",
                     help="skip the GEMM, flash-attention and batch-16 figures")
-    ap.add_argument("--design", choices=["gofilorn"],
-                    help="time this design beside the Llama decoder of equal size "
+    ap.add_argument("--design", choices=sorted(DESIGNS),
+                    help="time this design beside the closest decoder of equal size "
                          "instead of the headline workload")
     ap.add_argument("--design-size", choices=sorted(DESIGN_SIZES),
                     help="with --design: this size only")
-    ap.add_argument("--design-only", choices=["gofilorn", "llama"],
+    ap.add_argument("--design-only", choices=["gofilorn", "llama", "vamalix"],
                     help="with --design: this decoder only")
     args = ap.parse_args()
     if args.warmup < 3:

@@ -43,11 +43,14 @@ namespace {
     stop("vx_decoder: %s: %s", what, why);
 }
 
+/* Zeros. The decoder's stream does not wait for the one that the memset is queued on,
+   so it has to be over before anyone uses the memory. */
 template <typename T> T *dev_alloc(size_t count) {
   void *p = nullptr;
   if (cudaMalloc(&p, count * sizeof(T)) != cudaSuccess)
     stop("vx_decoder: out of device memory for %zu bytes", count * sizeof(T));
-  CUDA_OK(cudaMemset(p, 0, count * sizeof(T)));
+  CUDA_OK(cudaMemsetAsync(p, 0, count * sizeof(T), cudaStreamLegacy));
+  CUDA_OK(cudaStreamSynchronize(cudaStreamLegacy));
   return (T *)p;
 }
 

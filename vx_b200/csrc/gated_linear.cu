@@ -161,8 +161,6 @@ __global__ void __launch_bounds__(256)
 gated_linear_decay_kernel(const GatedLinearArgs a, const float *in, int64_t in_stride,
                           int t_count, float *alpha) {
   extern __shared__ __align__(16) float low[]; /* [TB][rank] */
-  chain_release();
-  chain_wait();
   const int t0 = blockIdx.x * TB, channels = a.heads * a.dim;
   const int a1 = Parts(a).a1;
   for (int i = threadIdx.x; i < TB * a.rank; i += 256) {
@@ -252,8 +250,6 @@ gated_linear_scan_kernel(const GatedLinearArgs a, const float *in, int64_t in_st
   const int step = 3 * dim + COLS; /* floats of a position: q | k | alpha | v */
   float *buf = scan_smem;          /* [2][TT][step] */
   float *so = buf + 2 * TT * step; /* [TT][COLS] */
-  chain_release();
-  chain_wait();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int h = blockIdx.y, col0 = blockIdx.x * COLS;
   const int g = lane % LG, group = lane / LG;
@@ -375,8 +371,6 @@ gated_linear_scan_kernel(const GatedLinearArgs a, const float *in, int64_t in_st
 __global__ void __launch_bounds__(256)
 gated_linear_finish_kernel(const GatedLinearArgs a, const float *in, int64_t in_stride,
                            const float *o, __nv_bfloat16 *terms, int cols) {
-  chain_release();
-  chain_wait();
   const int64_t t = blockIdx.x;
   const int lane = threadIdx.x & 31, gate = Parts(a).gate;
   for (int h = threadIdx.x >> 5; h < a.heads; h += 8) {
@@ -421,7 +415,7 @@ const char *launch_scan(const GatedLinearArgs &a, const float *in, int64_t in_st
   const void *kernel = (const void *)gated_linear_scan_kernel<LG, NI, RJ>;
   if (allow_dynamic_smem(kernel, most) != cudaSuccess)
     return "gated linear attention could not get its shared memory";
-  launch_chained(gated_linear_scan_kernel<LG, NI, RJ>,
+  launch_in_order(gated_linear_scan_kernel<LG, NI, RJ>,
                  dim3((a.vdim + COLS - 1) / COLS, a.heads), dim3(SCAN_THREADS), smem,
                  stream, a, in, in_stride, alpha, t, o);
   return check_launch("the recurrence of gated linear attention");
@@ -447,7 +441,7 @@ const char *gated_linear_decays(const GatedLinearArgs &a, const float *in,
                                 cudaStream_t stream) {
   if (const char *why = refuse(a, in_stride))
     return why;
-  launch_chained(gated_linear_decay_kernel,
+  launch_in_order(gated_linear_decay_kernel,
                  dim3((t + TB - 1) / TB, (a.heads * a.dim + 255) / 256), dim3(256),
                  TB * a.rank * sizeof(float), stream, a, in, in_stride, t, alpha);
   return check_launch("the decays of gated linear attention");
@@ -475,7 +469,7 @@ const char *gated_linear_finish(const GatedLinearArgs &a, const float *in,
     return why;
   if (cols % 4 != 0 || cols < a.heads * a.vdim)
     return "the output has too few columns";
-  launch_chained(gated_linear_finish_kernel, dim3(t), dim3(256), 0, stream, a, in,
+  launch_in_order(gated_linear_finish_kernel, dim3(t), dim3(256), 0, stream, a, in,
                  in_stride, o, (__nv_bfloat16 *)terms, cols);
   return check_launch("the norm and gate of gated linear attention");
 }

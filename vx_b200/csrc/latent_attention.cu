@@ -385,8 +385,6 @@ latent_down_kernel(const LatentArgs a, const float *partials, int splits, int t_
                    int q_rank, const float *q_gain, int q_mean, __nv_bfloat16 *terms) {
   extern __shared__ float down_row[]; /* [q_rank + kv_rank] */
   __shared__ float red[2][8];
-  chain_release();
-  chain_wait();
   const int64_t t = blockIdx.x;
   const int tid = threadIdx.x, K = a.kv_rank, both = q_rank + K, n = both + a.rot;
   const int pos = a.positions[0] + (int)t;
@@ -434,8 +432,6 @@ latent_down_kernel(const LatentArgs a, const float *partials, int splits, int t_
 __global__ void __launch_bounds__(256)
 latent_q_kernel(const LatentArgs a, const float *partials, int splits, int t_count,
                 float *q) {
-  chain_release();
-  chain_wait();
   const int hd = a.dim + a.rot, n = a.heads * hd;
   const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= (int64_t)t_count * (n / 4))
@@ -457,8 +453,6 @@ latent_q_kernel(const LatentArgs a, const float *partials, int splits, int t_cou
 /* a thread per (position, eight values of its latent) */
 __global__ void __launch_bounds__(256)
 latent_gather_kernel(const LatentArgs a, int first, int n, __nv_bfloat16 *terms) {
-  chain_release();
-  chain_wait();
   const int per_row = a.kv_rank / 8;
   const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= (int64_t)n * per_row)
@@ -494,8 +488,6 @@ latent_rows_kernel(const LatentArgs a, const float *q, const float *kv, int firs
   float (*sk)[KP + 4] = sq + AQ;
   float (*sv)[VP + 4] = reinterpret_cast<float (*)[VP + 4]>(sk + AK);
   float (*sp)[AK + 4] = reinterpret_cast<float (*)[AK + 4]>(sv + AK);
-  chain_release();
-  chain_wait();
   const int dim = a.dim, hd = a.dim + a.rot, vdim = a.vdim, head = blockIdx.y;
   const int t0 = blockIdx.x * AQ, base = a.positions[0];
   const int tid = threadIdx.x, ty = tid / 16, tx = tid % 16;
@@ -716,7 +708,7 @@ const char *launch_rows(const LatentArgs &a, const float *q, const float *kv, in
   if (allow_dynamic_smem((const void *)latent_rows_kernel<KP, VP, AQ, AK>, smem) !=
       cudaSuccess)
     return "the multi-position latent attention could not get its shared memory";
-  launch_chained(latent_rows_kernel<KP, VP, AQ, AK>, dim3((t + AQ - 1) / AQ, a.heads),
+  launch_in_order(latent_rows_kernel<KP, VP, AQ, AK>, dim3((t + AQ - 1) / AQ, a.heads),
                  dim3(ROW_THREADS), smem, stream, a, q, kv, first, t, terms, cols);
   return check_launch("the multi-position latent attention");
 }
@@ -746,7 +738,7 @@ const char *latent_rows_down(const LatentArgs &a, const float *partials, int spl
   if (smem > 200 * 1024 ||
       allow_dynamic_smem((const void *)latent_down_kernel, 200 * 1024) != cudaSuccess)
     return "the two latents of a position must fit in shared memory";
-  launch_chained(latent_down_kernel, dim3(t), dim3(256), smem, stream, a, partials, splits,
+  launch_in_order(latent_down_kernel, dim3(t), dim3(256), smem, stream, a, partials, splits,
                  t, q_rank, q_gain, q_mean, (__nv_bfloat16 *)terms);
   return check_launch("the latents of a prompt");
 }
@@ -756,7 +748,7 @@ const char *latent_rows_q(const LatentArgs &a, const float *partials, int splits
   if (const char *why = refuse(a))
     return why;
   const int64_t count = (int64_t)t * (a.heads * (a.dim + a.rot) / 4);
-  launch_chained(latent_q_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0,
+  launch_in_order(latent_q_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0,
                  stream, a, partials, splits, t, q);
   return check_launch("the queries of a prompt");
 }
@@ -766,7 +758,7 @@ const char *latent_rows_gather(const LatentArgs &a, int first, int n, void *term
   if (const char *why = refuse(a))
     return why;
   const int64_t count = (int64_t)n * (a.kv_rank / 8);
-  launch_chained(latent_gather_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0,
+  launch_in_order(latent_gather_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0,
                  stream, a, first, n, (__nv_bfloat16 *)terms);
   return check_launch("the latents of a window");
 }

@@ -82,7 +82,20 @@ cudaError_t launch_chained(void (*kernel)(KArgs...), dim3 grid, dim3 block,
   return cudaLaunchKernelEx(&cfg, kernel, std::forward<Args>(args)...);
 }
 
-/* The same for a kernel whose blocks form clusters of `cluster_x` along x
+/* In plain stream order: the kernel starts when the one before it has finished, and,
+   as long as it does not call chain_release(), the next one when it has. */
+template <typename... KArgs, typename... Args>
+cudaError_t launch_in_order(void (*kernel)(KArgs...), dim3 grid, dim3 block, size_t smem,
+                            cudaStream_t stream, Args &&...args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = grid;
+  cfg.blockDim = block;
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = stream;
+  return cudaLaunchKernelEx(&cfg, kernel, std::forward<Args>(args)...);
+}
+
+/* launch_chained for a kernel whose blocks form clusters of `cluster_x` along x
    (grid.x a multiple of it): the blocks of a cluster run together and can read
    one another's shared memory. */
 template <typename... KArgs, typename... Args>

@@ -48,8 +48,6 @@ streams_norm_kernel(void *out, const float *x, int64_t x_stride, const float *in
                     const NormGain w, int dim, float eps, const int32_t *pick) {
   extern __shared__ float u[]; /* [dim] */
   __shared__ float red[THREADS / 32];
-  chain_release();
-  chain_wait();
   const int64_t t = blockIdx.x;
   const float *xr = x + (pick ? pick[t] : t) * x_stride;
   float ss = 0.0f;
@@ -86,8 +84,6 @@ streams_mix_kernel(__nv_bfloat16 *terms, float *x, const float *partials, int sp
     sh.in[threadIdx.x] = next_in ? next_in[threadIdx.x] : 1.0f;
   }
   __syncthreads();
-  chain_release();
-  chain_wait();
   const int64_t t = blockIdx.x;
   float *xr = x + t * streams * (int64_t)dim;
   float ss = 0.0f;
@@ -124,8 +120,6 @@ streams_mix_kernel(__nv_bfloat16 *terms, float *x, const float *partials, int sp
 __global__ void __launch_bounds__(256)
 gelu_finish_kernel(__nv_bfloat16 *terms, const float *partials, int splits, int t_count,
                    int hidden) {
-  chain_release();
-  chain_wait();
   const int per_row = hidden / 8;
   const int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x;
   if (idx >= (int64_t)t_count * per_row)
@@ -158,7 +152,7 @@ const char *launch_norm(void *out, const float *x, int64_t x_stride, const Strea
   if (allow_dynamic_smem((const void *)streams_norm_kernel<TERMS>, 200 * 1024) !=
       cudaSuccess)
     return "the norm of the streams could not get its shared memory";
-  launch_chained(streams_norm_kernel<TERMS>, dim3(t), dim3(THREADS), dim * sizeof(float),
+  launch_in_order(streams_norm_kernel<TERMS>, dim3(t), dim3(THREADS), dim * sizeof(float),
                  stream, out, x, x_stride, m.in, m.streams, w, dim, eps, pick);
   return check_launch("the norm of the streams");
 }
@@ -169,7 +163,7 @@ const char *launch_mix(void *terms, float *x, const float *partials, int splits,
                        float eps, cudaStream_t stream) {
   if (allow_dynamic_smem((const void *)streams_mix_kernel<S>, 200 * 1024) != cudaSuccess)
     return "the mixing of the streams could not get its shared memory";
-  launch_chained(streams_mix_kernel<S>, dim3(t), dim3(THREADS), dim * sizeof(float),
+  launch_in_order(streams_mix_kernel<S>, dim3(t), dim3(THREADS), dim * sizeof(float),
                  stream, (__nv_bfloat16 *)terms, x, partials, splits, t, m, next_in, w,
                  dim, eps);
   return check_launch("the mixing of the streams");
@@ -216,7 +210,7 @@ const char *rows_gelu_finish(void *terms, const float *partials, int splits, int
   if (hidden % 8 != 0)
     return "the multi-position gelu takes a hidden size in multiples of 8";
   const int64_t count = (int64_t)t * (hidden / 8);
-  launch_chained(gelu_finish_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0,
+  launch_in_order(gelu_finish_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0,
                  stream, (__nv_bfloat16 *)terms, partials, splits, t, hidden);
   return check_launch("the multi-position gelu");
 }
