@@ -37,13 +37,15 @@ struct Parts {
 
 /* ---- one token of each sequence ------------------------------------------------
  * A cluster of CL blocks per (head, sequence), block r taking vdim / CL columns
- * (rounded up to 4). Threads: 8 groups of four columns by 32 rows. */
-constexpr int CL = 8, STEP_THREADS = 256, COLS4 = 8, ROWS = STEP_THREADS / COLS4;
+ * (rounded up to 4). Threads: COLS4 groups of four columns by ROWS rows. */
+constexpr int CL = 8, ROWS = 32;
 constexpr int EARLY = 8; /* rows of a thread that are fetched ahead of the wait */
 
-__global__ void __launch_bounds__(STEP_THREADS)
+template <int COLS4>
+__global__ void __launch_bounds__(COLS4 * ROWS)
 gated_linear_step_kernel(const GatedLinearArgs a, const float *in, int64_t in_stride,
                          float *out, int64_t out_stride) {
+  constexpr int STEP_THREADS = COLS4 * ROWS;
   extern __shared__ __align__(16) float step_smem[];
   const int slice4 = (a.vdim / 4 + CL - 1) / CL; /* float4 columns of a block */
   float *alpha = step_smem, *sk = alpha + a.dim, *sq = sk + a.dim; /* [dim] each */
@@ -198,9 +200,10 @@ gated_linear_decay_kernel(const GatedLinearArgs a, const float *in, int64_t in_s
  * LG lanes side by side hold the key channels of RJ columns (lane g of them channels
  * 4 (LG c + g) .. + 3, c below NI), so a warp holds 32 / LG * RJ columns of a head
  * and a block SCAN_WARPS times as many. q, k, alpha and v of TT positions at a time
- * come through two shared-memory buffers. Two columns go through a multiply-add
- * together. */
-constexpr int SCAN_WARPS = 4, SCAN_THREADS = SCAN_WARPS * 32, TT = 16;
+ * come through two shared-memory buffers (past the end: q = k = v = 0, alpha = 1, which
+ * leave the state as it is). Two channels go through a multiply-add together, and the
+ * sums over the lanes are taken for TS positions at once. */
+constexpr int SCAN_WARPS = 8, SCAN_THREADS = SCAN_WARPS * 32, TT = 16, TS = 8;
 
 __device__ __forceinline__ void copy16(float *dst, const float *src) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(ptx::smem_addr(dst)),
@@ -208,42 +211,42 @@ __device__ __forceinline__ void copy16(float *dst, const float *src) {
                : "memory");
 }
 
-/* The sums over the LG lanes of a group: half of the values change hands at every
-   exchange while there are several. Returns the one that this lane is left with;
-   `col` says which it is, `owner` whether this lane is to write it. */
-template <int LG, int RJ>
-__device__ __forceinline__ float group_sums(float (&v)[RJ], int g, int &col, bool &owner) {
-  col = 0;
+/* The sums of N values over the LG lanes of a group: half of the values change hands
+   at every exchange while there are several, so that lane g is left with the sums of
+   values first .. first + N / LG - 1 (N < LG: with value `first`, and the lowest of
+   the lanes that are writes it). */
+template <int LG, int N>
+__device__ __forceinline__ void group_sums(float (&v)[N], int g, int &first,
+                                           bool &owner) {
+  first = 0;
   owner = true;
-  int off = LG / 2;
+  int n = N;
 #pragma unroll
-  for (int n = RJ; n > 1; n /= 2) {
+  for (int off = LG / 2; off > 0; off /= 2) {
     const bool upper = (g & off) != 0;
+    if (n > 1) {
 #pragma unroll
-    for (int j = 0; j < RJ / 2; ++j)
-      if (j < n / 2) {
-        const float give = upper ? v[j] : v[j + n / 2];
-        const float keep = upper ? v[j + n / 2] : v[j];
-        v[j] = keep + __shfl_xor_sync(0xffffffffu, give, off);
-      }
-    if (upper)
-      col += n / 2;
-    off /= 2;
+      for (int j = 0; j < N / 2; ++j)
+        if (j < n / 2) {
+          const float give = upper ? v[j] : v[j + n / 2];
+          const float keep = upper ? v[j + n / 2] : v[j];
+          v[j] = keep + __shfl_xor_sync(0xffffffffu, give, off);
+        }
+      n /= 2;
+      if (upper)
+        first += n;
+    } else {
+      v[0] += __shfl_xor_sync(0xffffffffu, v[0], off);
+      owner = owner && !upper;
+    }
   }
-  float s = v[0];
-#pragma unroll
-  for (int rest = LG / 2 / RJ; rest > 0; rest /= 2) {
-    s += __shfl_xor_sync(0xffffffffu, s, rest);
-    owner = owner && (g & rest) == 0;
-  }
-  return s;
 }
 
 template <int LG, int NI, int RJ>
 __global__ void __launch_bounds__(SCAN_THREADS)
 gated_linear_scan_kernel(const GatedLinearArgs a, const float *in, int64_t in_stride,
                          const float *alpha, int t_count, float *o) {
-  static_assert(LG >= RJ && RJ >= 2, "a group has a lane for every column");
+  static_assert(RJ % 4 == 0 && TT % TS == 0, "columns in fours, whole batches");
   constexpr int WARP_COLS = 32 / LG * RJ, COLS = SCAN_WARPS * WARP_COLS;
   extern __shared__ __align__(16) float scan_smem[];
   const int dim = a.dim, vdim = a.vdim;
@@ -260,11 +263,15 @@ gated_linear_scan_kernel(const GatedLinearArgs a, const float *in, int64_t in_st
 
   auto fetch = [&](int t0, float *to) {
     const int quads = step / 4, dq = dim / 4, n = min(TT, t_count - t0);
-    for (int i = tid; i < n * quads; i += SCAN_THREADS) {
+    const int filled = (n + TS - 1) / TS * TS;
+    for (int i = tid; i < filled * quads; i += SCAN_THREADS) {
       const int t = i / quads, q = i - t * quads;
       const float *row = in + (int64_t)(t0 + t) * in_stride;
       float *dst = to + t * step + q * 4;
-      if (q < dq)
+      if (t >= n) {
+        const float v = q >= 2 * dq && q < 3 * dq ? 1.0f : 0.0f;
+        *reinterpret_cast<float4 *>(dst) = make_float4(v, v, v, v);
+      } else if (q < dq)
         copy16(dst, row + h * dim + q * 4);
       else if (q < 2 * dq)
         copy16(dst, row + at.k + h * dim + (q - dq) * 4);
@@ -279,19 +286,19 @@ gated_linear_scan_kernel(const GatedLinearArgs a, const float *in, int64_t in_st
     asm volatile("cp.async.commit_group;" ::: "memory");
   };
 
-  float2 s[4 * NI][RJ / 2];
+  float2 s[2 * NI][RJ]; /* two neighbouring channels of a column */
+  auto each_cell = [&](auto body) {
 #pragma unroll
-  for (int c = 0; c < NI; ++c)
+    for (int c = 0; c < 2 * NI; ++c)
 #pragma unroll
-    for (int e = 0; e < 4; ++e)
-#pragma unroll
-      for (int j = 0; j < RJ / 2; ++j) {
-        const int i = (c * LG + g) * 4 + e, col = col0 + mine + 2 * j;
-        s[c * 4 + e][j] = make_float2(0, 0);
-        if (!fresh && i < dim && col < vdim)
-          s[c * 4 + e][j] =
-              *reinterpret_cast<const float2 *>(state + (int64_t)i * vdim + col);
-      }
+      for (int j = 0; j < RJ; ++j)
+        body(s[c][j], ((c >> 1) * LG + g) * 4 + (c & 1) * 2, col0 + mine + j);
+  };
+  each_cell([&](float2 &cell, int i, int col) {
+    cell = make_float2(0, 0);
+    if (!fresh && i < dim && col < vdim)
+      cell = make_float2(state[(int64_t)i * vdim + col], state[(int64_t)(i + 1) * vdim + col]);
+  });
   fetch(0, buf);
   int side = 0;
   for (int t0 = 0; t0 < t_count; t0 += TT, side ^= 1) {
@@ -304,46 +311,55 @@ gated_linear_scan_kernel(const GatedLinearArgs a, const float *in, int64_t in_st
     }
     __syncthreads();
     const float *now = buf + side * TT * step;
-#pragma unroll 2
-    for (int t = 0; t < n; ++t, now += step) {
-      float2 v[RJ / 2], sum[RJ / 2];
+    for (int t = 0; t < n; t += TS) {
+      float part[TS * RJ];
 #pragma unroll
-      for (int j = 0; j < RJ / 2; ++j) {
-        v[j] = *reinterpret_cast<const float2 *>(now + 3 * dim + mine + 2 * j);
-        sum[j] = make_float2(0, 0);
-      }
+      for (int u = 0; u < TS; ++u, now += step) {
+        float v[RJ];
+        float2 sum[RJ];
 #pragma unroll
-      for (int c = 0; c < NI; ++c) {
-        const int i = (c * LG + g) * 4;
-        float4 q4 = make_float4(0, 0, 0, 0), k4 = q4, f4 = q4;
-        if (i < dim) {
-          q4 = *reinterpret_cast<const float4 *>(now + i);
-          k4 = *reinterpret_cast<const float4 *>(now + dim + i);
-          f4 = *reinterpret_cast<const float4 *>(now + 2 * dim + i);
+        for (int j = 0; j < RJ; j += 4) {
+          const float4 v4 = *reinterpret_cast<const float4 *>(now + 3 * dim + mine + j);
+          v[j] = v4.x; v[j + 1] = v4.y; v[j + 2] = v4.z; v[j + 3] = v4.w;
         }
-        const float q[4] = {q4.x, q4.y, q4.z, q4.w}, k[4] = {k4.x, k4.y, k4.z, k4.w},
-                    f[4] = {f4.x, f4.y, f4.z, f4.w};
 #pragma unroll
-        for (int e = 0; e < 4; ++e)
+        for (int j = 0; j < RJ; ++j)
+          sum[j] = make_float2(0, 0);
 #pragma unroll
-          for (int j = 0; j < RJ / 2; ++j) {
-            float2 &cell = s[c * 4 + e][j];
-            cell = mul_pair(make_float2(f[e], f[e]), cell);
-            fma_pair(cell, make_float2(k[e], k[e]), v[j]);
-            fma_pair(sum[j], make_float2(q[e], q[e]), cell);
+        for (int c = 0; c < NI; ++c) {
+          const int i = (c * LG + g) * 4;
+          float4 q = make_float4(0, 0, 0, 0), k = q, f = q;
+          if (i < dim) {
+            q = *reinterpret_cast<const float4 *>(now + i);
+            k = *reinterpret_cast<const float4 *>(now + dim + i);
+            f = *reinterpret_cast<const float4 *>(now + 2 * dim + i);
           }
-      }
-      float part[RJ];
 #pragma unroll
-      for (int j = 0; j < RJ / 2; ++j) {
-        part[2 * j] = sum[j].x;
-        part[2 * j + 1] = sum[j].y;
+          for (int e = 0; e < 2; ++e) {
+            const float2 q2 = e ? make_float2(q.z, q.w) : make_float2(q.x, q.y);
+            const float2 k2 = e ? make_float2(k.z, k.w) : make_float2(k.x, k.y);
+            const float2 f2 = e ? make_float2(f.z, f.w) : make_float2(f.x, f.y);
+#pragma unroll
+            for (int j = 0; j < RJ; ++j) {
+              float2 &cell = s[c * 2 + e][j];
+              cell = mul_pair(f2, cell);
+              fma_pair(cell, k2, make_float2(v[j], v[j]));
+              fma_pair(sum[j], q2, cell);
+            }
+          }
+        }
+#pragma unroll
+        for (int j = 0; j < RJ; ++j)
+          part[u * RJ + j] = sum[j].x + sum[j].y;
       }
-      int col;
+      int one;
       bool owner;
-      const float total = group_sums<LG, RJ>(part, g, col, owner);
+      group_sums<LG>(part, g, one, owner);
+      constexpr int LEFT = TS * RJ > LG ? TS * RJ / LG : 1;
       if (owner)
-        so[t * COLS + mine + col] = total * a.q_scale;
+#pragma unroll
+        for (int j = 0; j < LEFT; ++j)
+          so[(t + (one + j) / RJ) * COLS + mine + (one + j) % RJ] = part[j] * a.q_scale;
     }
     __syncthreads(); /* the buffer may be filled again; so is complete */
     for (int i = tid; i < n * (COLS / 4); i += SCAN_THREADS) {
@@ -354,16 +370,12 @@ gated_linear_scan_kernel(const GatedLinearArgs a, const float *in, int64_t in_st
             *reinterpret_cast<const float4 *>(&so[t * COLS + c]);
     }
   }
-#pragma unroll
-  for (int c = 0; c < NI; ++c)
-#pragma unroll
-    for (int e = 0; e < 4; ++e)
-#pragma unroll
-      for (int j = 0; j < RJ / 2; ++j) {
-        const int i = (c * LG + g) * 4 + e, col = col0 + mine + 2 * j;
-        if (i < dim && col < vdim)
-          *reinterpret_cast<float2 *>(state + (int64_t)i * vdim + col) = s[c * 4 + e][j];
-      }
+  each_cell([&](float2 &cell, int i, int col) {
+    if (i < dim && col < vdim) {
+      state[(int64_t)i * vdim + col] = cell.x;
+      state[(int64_t)(i + 1) * vdim + col] = cell.y;
+    }
+  });
 }
 
 /* ---- the positions of a prompt: norm and gate -----------------------------------
@@ -430,9 +442,14 @@ const char *gated_linear_decode(const GatedLinearArgs &a, const float *in,
     return why;
   const int slice4 = (a.vdim / 4 + CL - 1) / CL;
   const int smem = (3 * a.dim + slice4 * 4) * (int)sizeof(float);
-  launch_chained_cluster_smem(gated_linear_step_kernel, dim3(CL, a.heads, batch),
-                              dim3(STEP_THREADS), CL, smem, stream, a, in, in_stride, out,
-                              out_stride);
+  auto go = [&](auto kernel, int cols4) {
+    launch_chained_cluster_smem(kernel, dim3(CL, a.heads, batch), dim3(cols4 * ROWS), CL,
+                                smem, stream, a, in, in_stride, out, out_stride);
+  };
+  if (slice4 <= 8)
+    go(gated_linear_step_kernel<8>, 8);
+  else
+    go(gated_linear_step_kernel<16>, 16);
   return check_launch("a step of gated linear attention");
 }
 
@@ -452,13 +469,13 @@ const char *gated_linear_scan(const GatedLinearArgs &a, const float *in, int64_t
   if (const char *why = refuse(a, in_stride))
     return why;
   if (a.dim <= 32)
-    return launch_scan<8, 1, 8>(a, in, in_stride, alpha, t, o, stream);
+    return launch_scan<8, 1, 4>(a, in, in_stride, alpha, t, o, stream);
   if (a.dim <= 64)
-    return launch_scan<16, 1, 8>(a, in, in_stride, alpha, t, o, stream);
+    return launch_scan<16, 1, 4>(a, in, in_stride, alpha, t, o, stream);
   if (a.dim <= 128)
-    return launch_scan<32, 1, 8>(a, in, in_stride, alpha, t, o, stream);
+    return launch_scan<32, 1, 4>(a, in, in_stride, alpha, t, o, stream);
   if (a.dim <= 256)
-    return launch_scan<32, 2, 8>(a, in, in_stride, alpha, t, o, stream);
+    return launch_scan<32, 2, 4>(a, in, in_stride, alpha, t, o, stream);
   return launch_scan<32, 4, 4>(a, in, in_stride, alpha, t, o, stream);
 }
 

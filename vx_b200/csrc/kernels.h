@@ -571,6 +571,7 @@ struct LatentArgs {
 const char *latent_attention_decode(const LatentArgs &a, const float *q, int64_t q_stride,
                                     const float *down, int64_t down_stride, int batch,
                                     float *out, int64_t out_stride, cudaStream_t stream);
+int latent_status(); /* 0, or once the code of a copy that did not arrive */
 /* After the product with rows [q_rank | kv_rank | rot]: the normalised query latent
    as terms [t][3 q_rank], the ring's rows of the t positions. */
 const char *latent_rows_down(const LatentArgs &a, const float *partials, int splits, int t,

@@ -28,14 +28,19 @@ constexpr float LOWEST = -3.0e38f;
 /* ---- one new token per sequence ----------------------------------------------
  * A cluster of CL blocks per (sequence, tile of GH heads); block r takes the r-th run
  * of the window's positions and the r-th part of the two products' rows, its NW warps
- * every NW-th position, NB rows of the ring in flight per warp. A lane holds D4
- * float4s of a row. Warps and blocks meet in a fixed order. */
+ * every NW-th position. A warp's rows come through SLOTS shared-memory slots of its
+ * own, filled by bulk copies that it asks for ahead (all of them before the wait for
+ * the kernel in front, since earlier steps wrote them), NB rows at a time into
+ * registers, D4 float4s a lane. Warps and blocks meet in a fixed order. */
 constexpr int CL = 8;
+__host__ __device__ constexpr int row_slots(int D4) { return D4 <= 2 ? 8 : 4; }
 
 /* floats of dynamic shared memory */
 constexpr int latent_smem(int GH, int D4, int NW, int dim, int kv_rank) {
-  return (NW * GH + GH + 1) * D4 * 128 + GH * dim + GH * kv_rank / CL;
+  return (NW * row_slots(D4) + GH + 1) * D4 * 128 + GH * dim + GH * kv_rank / CL;
 }
+
+__device__ int g_latent_status; /* 0x61: a row of the ring never arrived */
 
 __device__ __forceinline__ float dot_word(const uint4 &w, const float *x,
                                           const __nv_bfloat16 *) {
@@ -58,71 +63,70 @@ __device__ __forceinline__ float dot_word(const uint4 &w, const float *x, const 
   return fmaf(__uint_as_float(w.w), a.w, s);
 }
 
-/* `tasks` dot products of `cols` values by a block's warps: row(i) is the weights of
-   task i, in(i) its input in shared memory, put(i, s) takes the result. As many lanes
-   as a row has words take one, U tasks of each such group are in flight. */
-template <typename W, int NW, typename Row, typename In, typename Put>
-__device__ __forceinline__ void block_dots(int tasks, int cols, Row row, In in, Put put) {
+/* y[r] = w[r] . x for `rows` rows of `cols` values, r taken in turn by the WARPS warps
+   of which this one is the `warp`-th; x in shared memory, put(r, y) takes a result. As
+   many lanes as a row has words take one, U rows of each such group are in flight. */
+template <typename W, int WARPS, typename Put>
+__device__ __forceinline__ void warp_dots(const W *w, int rows, int cols, const float *x,
+                                          int warp, Put put) {
   constexpr int E = 16 / (int)sizeof(W), U = 4;
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int lane = threadIdx.x & 31;
   const int words = cols / E;
   int lanes = 32;
   while (lanes > 1 && lanes / 2 >= words)
     lanes /= 2;
   const int groups = 32 / lanes, group = lane / lanes, first = lane % lanes;
-  for (int t0 = warp * groups * U; t0 < tasks; t0 += NW * groups * U) {
+  const int step = WARPS * groups;
+#pragma unroll 1
+  for (int r0 = warp * groups + group; r0 - group < rows; r0 += step * U) {
+    const uint4 *at = reinterpret_cast<const uint4 *>(w) + (int64_t)r0 * words;
     float s[U];
 #pragma unroll
     for (int u = 0; u < U; ++u)
       s[u] = 0.0f;
-#pragma unroll 2
+#pragma unroll 1
     for (int wd = first; wd < words; wd += lanes) {
-      uint4 w[U];
+      uint4 word[U];
 #pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const int i = t0 + u * groups + group;
-        w[u] = make_uint4(0, 0, 0, 0);
-        if (i < tasks)
-          w[u] = __ldg(reinterpret_cast<const uint4 *>(row(i)) + wd);
-      }
+      for (int u = 0; u < U; ++u)
+        word[u] = r0 + u * step < rows ? __ldg(at + u * step * words + wd)
+                                       : make_uint4(0, 0, 0, 0);
 #pragma unroll
-      for (int u = 0; u < U; ++u) {
-        const int i = t0 + u * groups + group;
-        if (i < tasks)
-          s[u] += dot_word(w[u], in(i) + wd * E, (const W *)nullptr);
-      }
+      for (int u = 0; u < U; ++u)
+        s[u] += dot_word(word[u], x + wd * E, (const W *)nullptr);
     }
     for (int o = lanes / 2; o > 0; o >>= 1)
 #pragma unroll
       for (int u = 0; u < U; ++u)
         s[u] += __shfl_xor_sync(0xffffffffu, s[u], o);
 #pragma unroll
-    for (int u = 0; u < U; ++u) {
-      const int i = t0 + u * groups + group;
-      if (first == 0 && i < tasks)
-        put(i, s[u]);
-    }
+    for (int u = 0; u < U; ++u)
+      if (first == 0 && r0 + u * step < rows)
+        put(r0 + u * step, s[u]);
   }
 }
 
 template <typename W, int GH, int D4, int NW>
-__global__ void __launch_bounds__(NW * 32)
+__global__ void __launch_bounds__(NW * 32, D4 <= 5 ? 2 : 1)
 latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
                      const float *down, int64_t down_stride, float *out,
                      int64_t out_stride) {
-  constexpr int NB = D4 == 1 ? 8 : D4 == 2 ? 4 : D4 <= 5 ? 2 : 1;
-  constexpr int THREADS = NW * 32, ROW = D4 * 128;
-  extern __shared__ __align__(16) float latent_shared[];
-  float *acc_s = latent_shared;         /* [NW][GH][ROW] */
-  float *heads_s = acc_s + NW * GH * ROW; /* [GH][ROW]: queries, then weighted latents */
+  constexpr int NB = D4 <= 2 ? 4 : D4 <= 5 ? 2 : 1;
+  constexpr int WPH = NW / GH; /* warps a head, in the two products */
+  constexpr int THREADS = NW * 32, ROW = D4 * 128, SLOTS = row_slots(D4);
+  extern __shared__ __align__(128) float latent_shared[];
+  float *slots_s = latent_shared; /* [NW][SLOTS][ROW]; the first GH then hold a warp's sums */
+  float *heads_s = slots_s + NW * SLOTS * ROW; /* [GH][ROW]: queries, then weighted latents */
   float *fresh = heads_s + GH * ROW;    /* [ROW]: this position's row */
   float *qn = fresh + ROW;              /* [GH][dim] */
   float *slice = qn + GH * a.dim;       /* [GH][kv_rank / CL] */
   __shared__ float warp_m[NW][GH], warp_l[NW][GH], red[NW];
   __shared__ float block_m[GH], block_l[GH], share[GH][CL];
+  __shared__ __align__(8) uint64_t bars[NW][SLOTS];
   cg::cluster_group cluster = cg::this_cluster();
   chain_release();
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  static_assert(GH <= SLOTS && NW % GH == 0, "a warp's sums fit its slots");
   const int rank = blockIdx.x, h0 = blockIdx.y * GH, b = blockIdx.z;
   const int nh = min(GH, a.heads - h0);
   const int K = a.kv_rank, part = K / CL, row_floats = K + a.rot;
@@ -152,33 +156,36 @@ latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
   for (int c = 0; c < D4; ++c)
     active[c] = (c * 32 + lane) * 4 < row_floats;
 
-  /* Rows below pos come from earlier steps; row pos is made here. */
-  float4 kv[NB][D4];
-  auto load = [&](int t0, bool own) {
-#pragma unroll
-    for (int j = 0; j < NB; ++j) {
-      const int t = t0 + j * NW;
-      if (t >= t_end || (t == pos) != own)
-        continue;
-      int row = row_low + (t - low);
-      if (row >= a.cache_rows)
-        row -= a.cache_rows;
-      const float *src = own ? fresh : ring + (int64_t)row * row_floats;
-#pragma unroll
-      for (int c = 0; c < D4; ++c)
-        if (active[c])
-          kv[j][c] = *reinterpret_cast<const float4 *>(src + (c * 32 + lane) * 4);
-    }
+  /* Rows below pos come from earlier steps; row pos is made here. This warp's rows are
+     t_begin + warp + j NW, `have` of them in the ring. */
+  const int mine = t_begin + warp;
+  const int have = max(0, (min(t_end, pos) - mine + NW - 1) / NW);
+  float *my_slots = slots_s + warp * SLOTS * ROW;
+  auto ask = [&](int j) { /* lane 0 */
+    int row = row_low + (mine + j * NW - low);
+    if (row >= a.cache_rows)
+      row -= a.cache_rows;
+    uint64_t *bar = &bars[warp][j % SLOTS];
+    ptx::mbar_expect_tx(bar, row_floats * (int)sizeof(float));
+    ptx::bulk_load(my_slots + j % SLOTS * ROW, ring + (int64_t)row * row_floats,
+                   row_floats * (int)sizeof(float), bar);
   };
-#pragma unroll
-  for (int j = 0; j < NB; ++j)
-#pragma unroll
-    for (int c = 0; c < D4; ++c)
-      kv[j][c] = make_float4(0, 0, 0, 0);
-  load(t_begin + warp, false);
+  if (lane == 0) {
+    for (int k = 0; k < SLOTS; ++k)
+      ptx::mbar_init(&bars[warp][k], 1);
+    ptx::fence_proxy_async_smem();
+    ptx::fence_barrier_init();
+    for (int j = 0; j < min(SLOTS, have); ++j)
+      ask(j);
+  }
+  __syncwarp();
   chain_wait();
 
-  /* ---- this position's row; the queries, rotated ---- */
+  /* ---- this position's row; the queries, rotated; what fills rows up ---- */
+  for (int i = row_floats + tid; i < ROW; i += THREADS)
+#pragma unroll
+    for (int h = 0; h <= GH; ++h) /* fresh follows the heads */
+      heads_s[h * ROW + i] = 0.0f;
   const float *dn = down + b * down_stride;
   const float *q = q_in + b * q_stride + (int64_t)h0 * (a.dim + a.rot);
   float ss = 0.0f;
@@ -214,10 +221,10 @@ latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
     fresh[i] = fresh[i] * inv * a.gain[i];
 
   /* ---- the queries for latents: this block's part of each, then all parts ---- */
-  block_dots<W, NW>(
-      nh * part, a.dim, [&](int i) { return uk_row(i / part, i % part); },
-      [&](int i) { return qn + i / part * a.dim; },
-      [&](int i, float s) { slice[i] = s; });
+  const int g_mine = warp % GH; /* the head whose products this warp takes part in */
+  if (g_mine < nh)
+    warp_dots<W, WPH>(uk_row(g_mine, 0), part, a.dim, qn + g_mine * a.dim, warp / GH,
+                      [&](int r, float y) { slice[g_mine * part + r] = y; });
   auto gather = [&] {
     for (int i = tid; i < nh * K / 4; i += THREADS) {
       const int g = i / (K / 4), c = (i - g * (K / 4)) * 4, r = c / part;
@@ -234,67 +241,103 @@ latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
     for (int i = tid; i < row_floats; i += THREADS)
       to[i] = fresh[i];
   }
-  load(t_begin + warp, true);
-
-  float4 qr[GH][D4], acc[GH][D4];
+  float2 acc[GH][D4][2];
   float m[GH], l[GH];
 #pragma unroll
   for (int h = 0; h < GH; ++h) {
     m[h] = LOWEST;
     l[h] = 0.0f;
 #pragma unroll
-    for (int c = 0; c < D4; ++c) {
-      acc[h][c] = qr[h][c] = make_float4(0, 0, 0, 0);
-      if (active[c] && h < nh)
-        qr[h][c] =
-            *reinterpret_cast<const float4 *>(heads_s + h * ROW + (c * 32 + lane) * 4);
-    }
+    for (int c = 0; c < D4; ++c)
+      acc[h][c][0] = acc[h][c][1] = make_float2(0, 0);
   }
-  for (int t0 = t_begin + warp; t0 < t_end; t0 += NB * NW) {
-    if (t0 != t_begin + warp) {
-      load(t0, false);
-      load(t0, true);
+  bool arrived = true;
+  for (int j0 = 0; mine + j0 * NW < t_end; j0 += NB) {
+    const int t0 = mine + j0 * NW;
+    float4 kv[NB][D4];
+#pragma unroll
+    for (int k = 0; k < NB; ++k) {
+      const int j = j0 + k, slot = j % SLOTS;
+      const float *src = fresh;
+      if (j < have) {
+        uint64_t *bar = &bars[warp][slot];
+        const uint32_t phase = (j / SLOTS) & 1;
+        arrived = arrived &&
+                  (ptx::mbar_try_wait(bar, phase) || ptx::mbar_wait_alone(bar, phase));
+        src = my_slots + slot * ROW;
+      }
+#pragma unroll
+      for (int c = 0; c < D4; ++c)
+        kv[k][c] = active[c] && t0 + k * NW < t_end
+                       ? *reinterpret_cast<const float4 *>(src + (c * 32 + lane) * 4)
+                       : make_float4(0, 0, 0, 0);
     }
+    if (!arrived) {
+      atomicCAS(&g_latent_status, 0, 0x61);
+      for (int j = j0; j < min(j0 + SLOTS, have); ++j) /* what is still on its way */
+        ptx::mbar_wait_alone(&bars[warp][j % SLOTS], (j / SLOTS) & 1);
+      break;
+    }
+    __syncwarp(); /* every lane has the rows: their slots may be filled again */
+    if (lane == 0)
+      for (int j = j0 + SLOTS; j < min(j0 + NB + SLOTS, have); ++j)
+        ask(j);
+    float s[GH][NB];
 #pragma unroll
     for (int h = 0; h < GH; ++h) {
-      float s[NB];
+      float2 d[NB];
 #pragma unroll
-      for (int j = 0; j < NB; ++j) {
-        s[j] = 0.0f;
+      for (int k = 0; k < NB; ++k)
+        d[k] = make_float2(0, 0);
 #pragma unroll
-        for (int c = 0; c < D4; ++c) {
-          s[j] = fmaf(qr[h][c].x, kv[j][c].x, s[j]);
-          s[j] = fmaf(qr[h][c].y, kv[j][c].y, s[j]);
-          s[j] = fmaf(qr[h][c].z, kv[j][c].z, s[j]);
-          s[j] = fmaf(qr[h][c].w, kv[j][c].w, s[j]);
+      for (int c = 0; c < D4; ++c) {
+        const float4 q4 =
+            *reinterpret_cast<const float4 *>(heads_s + h * ROW + (c * 32 + lane) * 4);
+#pragma unroll
+        for (int k = 0; k < NB; ++k) {
+          fma_pair(d[k], make_float2(q4.x, q4.y), make_float2(kv[k][c].x, kv[k][c].y));
+          fma_pair(d[k], make_float2(q4.z, q4.w), make_float2(kv[k][c].z, kv[k][c].w));
         }
       }
 #pragma unroll
-      for (int o = 16; o > 0; o >>= 1)
+      for (int k = 0; k < NB; ++k)
+        s[h][k] = d[k].x + d[k].y;
+    }
 #pragma unroll
-        for (int j = 0; j < NB; ++j)
-          s[j] += __shfl_xor_sync(0xffffffffu, s[j], o);
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+      for (int h = 0; h < GH; ++h)
+#pragma unroll
+        for (int k = 0; k < NB; ++k)
+          s[h][k] += __shfl_xor_sync(0xffffffffu, s[h][k], o);
+#pragma unroll
+    for (int h = 0; h < GH; ++h) {
       float big = m[h];
 #pragma unroll
-      for (int j = 0; j < NB; ++j) {
-        s[j] = t0 + j * NW < t_end ? s[j] * a.scale : LOWEST;
-        big = fmaxf(big, s[j]);
+      for (int k = 0; k < NB; ++k) {
+        s[h][k] = t0 + k * NW < t_end ? s[h][k] * a.scale : LOWEST;
+        big = fmaxf(big, s[h][k]);
       }
       const float fix = expf(m[h] - big);
       m[h] = big;
       l[h] *= fix;
+      float w[NB];
 #pragma unroll
-      for (int c = 0; c < D4; ++c) {
-        acc[h][c].x *= fix; acc[h][c].y *= fix;
-        acc[h][c].z *= fix; acc[h][c].w *= fix;
+      for (int k = 0; k < NB; ++k) {
+        w[k] = t0 + k * NW < t_end ? expf(s[h][k] - big) : 0.0f;
+        l[h] += w[k];
       }
 #pragma unroll
-      for (int j = 0; j < NB; ++j) {
-        const float w = t0 + j * NW < t_end ? expf(s[j] - big) : 0.0f;
-        l[h] += w;
+      for (int c = 0; c < D4; ++c) {
+        acc[h][c][0] = mul_pair(acc[h][c][0], make_float2(fix, fix));
+        acc[h][c][1] = mul_pair(acc[h][c][1], make_float2(fix, fix));
 #pragma unroll
-        for (int c = 0; c < D4; ++c)
-          axpy(acc[h][c], w, kv[j][c]);
+        for (int k = 0; k < NB; ++k) {
+          fma_pair(acc[h][c][0], make_float2(w[k], w[k]),
+                   make_float2(kv[k][c].x, kv[k][c].y));
+          fma_pair(acc[h][c][1], make_float2(w[k], w[k]),
+                   make_float2(kv[k][c].z, kv[k][c].w));
+        }
       }
     }
   }
@@ -308,8 +351,8 @@ latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
     }
 #pragma unroll
     for (int c = 0; c < D4; ++c)
-      *reinterpret_cast<float4 *>(acc_s + (warp * GH + h) * ROW + (c * 32 + lane) * 4) =
-          acc[h][c];
+      *reinterpret_cast<float4 *>(my_slots + h * ROW + (c * 32 + lane) * 4) =
+          make_float4(acc[h][c][0].x, acc[h][c][0].y, acc[h][c][1].x, acc[h][c][1].y);
   }
   __syncthreads();
   for (int i = warp; i < nh * D4; i += NW) {
@@ -323,10 +366,10 @@ latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
       const float f = expf(warp_m[w][h] - big);
       sum = fmaf(f, warp_l[w][h], sum);
       axpy(o, f,
-           *reinterpret_cast<const float4 *>(acc_s + (w * GH + h) * ROW +
+           *reinterpret_cast<const float4 *>(slots_s + (w * SLOTS + h) * ROW +
                                              (c * 32 + lane) * 4));
     }
-    *reinterpret_cast<float4 *>(acc_s + h * ROW + (c * 32 + lane) * 4) = o;
+    *reinterpret_cast<float4 *>(slots_s + h * ROW + (c * 32 + lane) * 4) = o;
     if (lane == 0 && c == 0) {
       block_m[h] = big;
       block_l[h] = sum;
@@ -358,7 +401,7 @@ latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
 #pragma unroll
     for (int r = 0; r < CL; ++r)
       axpy(o, share[g][r],
-           *reinterpret_cast<const float4 *>(cluster.map_shared_rank(acc_s, r) + g * ROW +
+           *reinterpret_cast<const float4 *>(cluster.map_shared_rank(slots_s, r) + g * ROW +
                                              rank * part + c));
     *reinterpret_cast<float4 *>(slice + g * part + c) = o;
   }
@@ -368,13 +411,11 @@ latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
   __syncthreads();
 
   /* ---- through the value matrix ---- */
-  if (vn > 0)
-    block_dots<W, NW>(
-        nh * vn, K, [&](int i) { return uv_row(i / vn, i % vn); },
-        [&](int i) { return heads_s + i / vn * ROW; },
-        [&](int i, float s) {
-          out[b * out_stride + (int64_t)(h0 + i / vn) * a.vdim + v0 + i % vn] = s;
-        });
+  if (vn > 0 && g_mine < nh)
+    warp_dots<W, WPH>(uv_row(g_mine, 0), vn, K, heads_s + g_mine * ROW, warp / GH,
+                      [&](int r, float y) {
+                        out[b * out_stride + (int64_t)(h0 + g_mine) * a.vdim + v0 + r] = y;
+                      });
   cluster.barrier_wait();
 }
 
@@ -663,31 +704,59 @@ struct StepCall {
   cudaStream_t stream;
 };
 
-template <typename W, int GH, int D4>
-const char *launch_step(const LatentArgs &a, const StepCall &c) {
-  constexpr int NW = 8;
-  const int smem = latent_smem(GH, D4, NW, a.dim, a.kv_rank) * (int)sizeof(float);
-  constexpr int most = latent_smem(GH, D4, NW, 512, D4 * 128) * (int)sizeof(float);
-  static_assert(most <= 200 * 1024, "the arrays fit in shared memory");
-  if (allow_dynamic_smem((const void *)latent_decode_kernel<W, GH, D4, NW>, most) !=
-      cudaSuccess)
-    return "latent attention could not get its shared memory";
-  launch_chained_cluster_smem(latent_decode_kernel<W, GH, D4, NW>,
-                              dim3(CL, (a.heads + GH - 1) / GH, c.batch), dim3(NW * 32),
-                              CL, smem, c.stream, a, c.q, c.q_stride, c.down,
-                              c.down_stride, c.out, c.out_stride);
-  return check_launch("a step of latent attention");
-}
+template <typename W, int GH, int D4> struct Step {
+  static constexpr int NW = 8;
+  static constexpr int most = latent_smem(GH, D4, NW, 512, D4 * 128) * (int)sizeof(float);
+  static_assert(most <= 226 * 1024, "the arrays fit in shared memory");
+
+  static int smem(const LatentArgs &a) {
+    return latent_smem(GH, D4, NW, a.dim, a.kv_rank) * (int)sizeof(float);
+  }
+  static bool allowed() {
+    return allow_dynamic_smem((const void *)latent_decode_kernel<W, GH, D4, NW>, most) ==
+           cudaSuccess;
+  }
+  /* whether the clusters all run at once */
+  static bool one_wave(const LatentArgs &a, int batch) {
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(CL, (a.heads + GH - 1) / GH, batch);
+    cfg.blockDim = dim3(NW * 32);
+    cfg.dynamicSmemBytes = smem(a);
+    cudaLaunchAttribute attr[1];
+    attr[0].id = cudaLaunchAttributeClusterDimension;
+    attr[0].val.clusterDim.x = CL;
+    attr[0].val.clusterDim.y = 1;
+    attr[0].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = 1;
+    int clusters = 0;
+    if (!allowed() || cudaOccupancyMaxActiveClusters(
+                          &clusters, latent_decode_kernel<W, GH, D4, NW>, &cfg) !=
+                          cudaSuccess) {
+      cudaGetLastError();
+      return false;
+    }
+    return (int64_t)cfg.gridDim.y * batch <= clusters;
+  }
+  static const char *launch(const LatentArgs &a, const StepCall &c) {
+    if (!allowed())
+      return "latent attention could not get its shared memory";
+    launch_chained_cluster_smem(latent_decode_kernel<W, GH, D4, NW>,
+                                dim3(CL, (a.heads + GH - 1) / GH, c.batch), dim3(NW * 32),
+                                CL, smem(a), c.stream, a, c.q, c.q_stride, c.down,
+                                c.down_stride, c.out, c.out_stride);
+    return check_launch("a step of latent attention");
+  }
+};
 
 template <typename W, int D4>
 const char *launch_step_heads(const LatentArgs &a, const StepCall &c) {
-  /* as many heads a cluster as keep the grid within one wave */
-  const int64_t clusters = (int64_t)a.heads * c.batch;
-  if (clusters * CL <= sm_count())
-    return launch_step<W, 1, D4>(a, c);
-  if (D4 > 2 || clusters * CL <= 2 * sm_count())
-    return launch_step<W, 2, D4>(a, c);
-  return launch_step<W, (D4 > 2 ? 2 : 4), D4>(a, c);
+  /* few heads a cluster as long as the clusters all run at once */
+  if ((int64_t)a.heads * c.batch * CL <= sm_count() && Step<W, 1, D4>::one_wave(a, c.batch))
+    return Step<W, 1, D4>::launch(a, c);
+  if (D4 > 2 || Step<W, 2, D4>::one_wave(a, c.batch))
+    return Step<W, 2, D4>::launch(a, c);
+  return Step<W, (D4 > 2 ? 2 : 4), D4>::launch(a, c);
 }
 
 template <typename W> const char *launch_step_row(const LatentArgs &a, const StepCall &c) {
@@ -727,6 +796,15 @@ const char *latent_attention_decode(const LatentArgs &a, const float *q, int64_t
   const StepCall c{q, q_stride, down, down_stride, batch, out, out_stride, stream};
   return a.fmt == kFmtBf16 ? launch_step_row<__nv_bfloat16>(a, c)
                            : launch_step_row<float>(a, c);
+}
+
+int latent_status() {
+  int v = 0, zero = 0;
+  if (cudaMemcpyFromSymbol(&v, g_latent_status, sizeof v) != cudaSuccess)
+    return -1;
+  if (v)
+    cudaMemcpyToSymbol(g_latent_status, &zero, sizeof zero);
+  return v;
 }
 
 const char *latent_rows_down(const LatentArgs &a, const float *partials, int splits, int t,

@@ -1096,7 +1096,8 @@ int32_t vx_b200_kernel_status(void) {
   const int r = vxb::rows_status();
   const int s = vxb::step_status(vxb::caller_stream());
   const int e = vxb::moe_group_status(vxb::caller_stream());
-  return g ? g : (f ? f : (t ? t : (m ? m : (r ? r : (s ? s : e)))));
+  const int l = vxb::latent_status();
+  return g ? g : (f ? f : (t ? t : (m ? m : (r ? r : (s ? s : (e ? e : l))))));
 }
 
 int32_t vx_b200_attention_kernel(int32_t which) {

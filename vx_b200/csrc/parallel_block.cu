@@ -128,6 +128,21 @@ sum_kernel(float *out, const float *partials, int splits, int t_count, int n, fl
                           cap);
 }
 
+/* The same for n a multiple of 4, four values a thread. */
+__global__ void __launch_bounds__(256)
+sum4_kernel(float *out, const float *partials, int splits, int t_count, int n, float scale,
+            float cap) {
+  chain_release();
+  chain_wait();
+  const int64_t idx = ((int64_t)blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (idx >= (int64_t)t_count * n)
+    return;
+  const float4 s = sum_runs4(partials, splits, 1, (int64_t)t_count * n, 0, idx);
+  *reinterpret_cast<float4 *>(out + idx) =
+      make_float4(capped_logit(s.x, scale, cap), capped_logit(s.y, scale, cap),
+                  capped_logit(s.z, scale, cap), capped_logit(s.w, scale, cap));
+}
+
 /* ---- the f32 product on the FP32 pipe: 64 positions x 64 rows a block, 4 x 4 a
    thread, the terms added up again (exactly) on their way into shared memory --- */
 constexpr int GT = 64, GC = 16;
@@ -218,8 +233,12 @@ const char *rows_fan_finish(const float *partials, int splits, int t, int n,
 const char *rows_sum(float *out, const float *partials, int splits, int t, int n,
                      cudaStream_t stream, float scale, float cap) {
   const int64_t count = (int64_t)t * n;
-  launch_chained(sum_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0, stream,
-                 out, partials, splits, t, n, scale, cap);
+  if (n % 4 == 0)
+    launch_chained(sum4_kernel, dim3((unsigned)((count / 4 + 255) / 256)), dim3(256), 0,
+                   stream, out, partials, splits, t, n, scale, cap);
+  else
+    launch_chained(sum_kernel, dim3((unsigned)((count + 255) / 256)), dim3(256), 0,
+                   stream, out, partials, splits, t, n, scale, cap);
   return check_launch("the sum of a product's runs");
 }
 

@@ -3,9 +3,8 @@
  * output, which the norm of the next sublayer follows in the same pass.  (A step has
  * both inside its projections: stream_proj.)
  *
- * A block is a position; thread i keeps values i, i + 256, ... of every stream to
- * itself, so the streams of a position are read once, mixed in registers and written
- * once.
+ * A block is a position; a thread keeps its values of every stream to itself, so the
+ * streams of a position are read once, mixed in registers and written once.
  */
 #include "kernels.h"
 #include "launch.cuh"
@@ -46,74 +45,100 @@ __global__ void __launch_bounds__(THREADS)
 streams_norm_kernel(void *out, const float *x, int64_t x_stride, const float *in,
                     int streams,
                     const NormGain w, int dim, float eps, const int32_t *pick) {
-  extern __shared__ float u[]; /* [dim] */
+  extern __shared__ __align__(16) float u[]; /* [dim] */
   __shared__ float red[THREADS / 32];
   const int64_t t = blockIdx.x;
   const float *xr = x + (pick ? pick[t] : t) * x_stride;
   float ss = 0.0f;
-  for (int i = threadIdx.x; i < dim; i += THREADS) {
-    float v = 0.0f;
+  for (int i = threadIdx.x * 4; i < dim; i += THREADS * 4) {
+    float4 v = make_float4(0, 0, 0, 0);
+#pragma unroll 4
     for (int s = 0; s < streams; ++s)
-      v = fmaf(in ? in[s] : 1.0f, xr[(int64_t)s * dim + i], v);
-    u[i] = v;
-    ss = fmaf(v, v, ss);
+      axpy(v, in ? in[s] : 1.0f,
+           *reinterpret_cast<const float4 *>(xr + (int64_t)s * dim + i));
+    *reinterpret_cast<float4 *>(u + i) = v;
+    ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
   }
   const float inv = block_rms(ss, w.n ? w.n : dim, eps, red);
-  for (int i = threadIdx.x; i < dim; i += THREADS) {
-    const float v = u[i] * gain_of(w, i) * inv;
+  for (int i = threadIdx.x * 4; i < dim; i += THREADS * 4) {
+    const float4 v = *reinterpret_cast<const float4 *>(u + i);
+    const float n[4] = {v.x * gain_of(w, i) * inv, v.y * gain_of(w, i + 1) * inv,
+                        v.z * gain_of(w, i + 2) * inv, v.w * gain_of(w, i + 3) * inv};
     if (TERMS)
-      store_terms((__nv_bfloat16 *)out, dim, t, i, v);
+      store_terms4((__nv_bfloat16 *)out, dim, t, i, n);
     else
-      ((float *)out)[t * dim + i] = v;
+      *reinterpret_cast<float4 *>((float *)out + t * dim + i) =
+          make_float4(n[0], n[1], n[2], n[3]);
   }
 }
 
-/* S: the number of streams, or 0 for any. */
+/* S streams, a thread four neighbouring values of all of them at a time; S 0: any
+   number, a value at a time. */
 template <int S>
 __global__ void __launch_bounds__(THREADS)
 streams_mix_kernel(__nv_bfloat16 *terms, float *x, const float *partials, int splits,
                    int t_count, const StreamMix m, const float *next_in,
                    const NormGain w, int dim, float eps) {
-  extern __shared__ float u[]; /* [dim] */
+  extern __shared__ __align__(16) float u[]; /* [dim], S 0: then [streams][THREADS] */
   __shared__ MixShared sh;
-  const int streams = S ? S : m.streams;
-  for (int i = threadIdx.x; i < streams * streams; i += THREADS)
+  const int streams = S ? S : m.streams, tid = threadIdx.x;
+  for (int i = tid; i < streams * streams; i += THREADS)
     sh.mix[i] = m.mix[i];
-  if ((int)threadIdx.x < streams) {
-    sh.out[threadIdx.x] = m.out[threadIdx.x];
-    sh.in[threadIdx.x] = next_in ? next_in[threadIdx.x] : 1.0f;
+  if (tid < streams) {
+    sh.out[tid] = m.out[tid];
+    sh.in[tid] = next_in ? next_in[tid] : 1.0f;
   }
   __syncthreads();
   const int64_t t = blockIdx.x;
   float *xr = x + t * streams * (int64_t)dim;
   float ss = 0.0f;
-  for (int i = threadIdx.x; i < dim; i += THREADS) {
-    const float y = sum_runs(partials, splits, t_count, dim, t, i);
-    float old[S ? S : kMaxStreams], v = 0.0f;
+  if constexpr (S > 0) {
+    for (int i = tid * 4; i < dim; i += THREADS * 4) {
+      float4 old[S], v = make_float4(0, 0, 0, 0);
 #pragma unroll
-    for (int s = 0; s < (S ? S : kMaxStreams); ++s)
-      if (S || s < streams)
-        old[s] = xr[(int64_t)s * dim + i];
+      for (int s = 0; s < S; ++s)
+        old[s] = *reinterpret_cast<const float4 *>(xr + (int64_t)s * dim + i);
+      const float4 y = sum_runs4(partials, splits, t_count, dim, t, i);
 #pragma unroll
-    for (int to = 0; to < (S ? S : kMaxStreams); ++to) {
-      if (!S && to >= streams)
-        break;
-      float now = sh.out[to] * y;
+      for (int to = 0; to < S; ++to) {
+        float4 now = make_float4(0, 0, 0, 0);
+        axpy(now, sh.out[to], y);
 #pragma unroll
-      for (int s = 0; s < (S ? S : kMaxStreams); ++s)
-        if (S || s < streams)
-          now = fmaf(sh.mix[s * streams + to], old[s], now);
-      xr[(int64_t)to * dim + i] = now;
-      v = fmaf(sh.in[to], now, v);
+        for (int s = 0; s < S; ++s)
+          axpy(now, sh.mix[s * S + to], old[s]);
+        *reinterpret_cast<float4 *>(xr + (int64_t)to * dim + i) = now;
+        axpy(v, sh.in[to], now);
+      }
+      *reinterpret_cast<float4 *>(u + i) = v;
+      ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
     }
-    u[i] = v;
-    ss = fmaf(v, v, ss);
+  } else {
+    float *old = u + dim;
+    for (int i = tid; i < dim; i += THREADS) {
+      const float y = sum_runs(partials, splits, t_count, dim, t, i);
+      float v = 0.0f;
+      for (int s = 0; s < streams; ++s)
+        old[s * THREADS + tid] = xr[(int64_t)s * dim + i];
+      for (int to = 0; to < streams; ++to) {
+        float now = sh.out[to] * y;
+        for (int s = 0; s < streams; ++s)
+          now = fmaf(sh.mix[s * streams + to], old[s * THREADS + tid], now);
+        xr[(int64_t)to * dim + i] = now;
+        v = fmaf(sh.in[to], now, v);
+      }
+      u[i] = v;
+      ss = fmaf(v, v, ss);
+    }
   }
   if (!terms)
     return;
-  const float inv = block_rms(ss, w.n ? w.n : dim, eps, sh.red);
-  for (int i = threadIdx.x; i < dim; i += THREADS)
-    store_terms(terms, dim, t, i, u[i] * gain_of(w, i) * inv);
+  const float inv = block_rms(ss, w.n ? w.n : dim, eps, sh.red); /* u is complete */
+  for (int i = tid * 4; i < dim; i += THREADS * 4) {
+    const float4 v = *reinterpret_cast<const float4 *>(u + i);
+    const float n[4] = {v.x * gain_of(w, i) * inv, v.y * gain_of(w, i + 1) * inv,
+                        v.z * gain_of(w, i + 2) * inv, v.w * gain_of(w, i + 3) * inv};
+    store_terms4(terms, dim, t, i, n);
+  }
 }
 
 /* a thread per (position, eight rows) */
@@ -161,10 +186,12 @@ template <int S>
 const char *launch_mix(void *terms, float *x, const float *partials, int splits, int t,
                        const StreamMix &m, const float *next_in, NormGain w, int dim,
                        float eps, cudaStream_t stream) {
-  if (allow_dynamic_smem((const void *)streams_mix_kernel<S>, 200 * 1024) != cudaSuccess)
+  const size_t smem = (dim + (S ? 0 : m.streams * THREADS)) * sizeof(float);
+  if (smem > 216 * 1024 || dim % 4 != 0)
+    return "the streams of a position must fit in shared memory";
+  if (allow_dynamic_smem((const void *)streams_mix_kernel<S>, 216 * 1024) != cudaSuccess)
     return "the mixing of the streams could not get its shared memory";
-  launch_in_order(streams_mix_kernel<S>, dim3(t), dim3(THREADS), dim * sizeof(float),
-                 stream, (__nv_bfloat16 *)terms, x, partials, splits, t, m, next_in, w,
+  launch_in_order(streams_mix_kernel<S>, dim3(t), dim3(THREADS), smem, stream, (__nv_bfloat16 *)terms, x, partials, splits, t, m, next_in, w,
                  dim, eps);
   return check_launch("the mixing of the streams");
 }

@@ -334,40 +334,71 @@ rowdot_kernel(const RowDotParams p) {
          projection. */
       const float4 *px4 = reinterpret_cast<const float4 *>(px);
       const int quads = cols / 4;
-      for (int q0 = threadIdx.x; q0 < quads; q0 += 4 * blockDim.x) {
-        float4 v[4], wn[4];
+      auto gains = [&](int q) {
+        if (p.norm_bf16) {
+          const uint2 w = reinterpret_cast<const uint2 *>(p.norm_w)[q];
+          return make_float4(bf_lo(w.x), bf_hi(w.x), bf_lo(w.y), bf_hi(w.y));
+        }
+        return reinterpret_cast<const float4 *>(p.norm_w)[q];
+      };
+      auto stage = [&](int q, const float4 &v, const float4 &wn) {
+        *reinterpret_cast<float4 *>(&xs[b * xs_stride + xs_at(4 * q)]) =
+            make_float4(v.x * wn.x, v.y * wn.y, v.z * wn.z, v.w * wn.w);
+        ss = fmaf(v.x, v.x, ss);
+        ss = fmaf(v.y, v.y, ss);
+        ss = fmaf(v.z, v.z, ss);
+        ss = fmaf(v.w, v.w, ss);
+      };
+      if constexpr (reads_streams(EPI)) {
+        /* the weighted sum of the streams takes the place of x: two quads of four
+           streams in flight */
+        const int64_t next = p.stream_stride / 4;
+        for (int q0 = threadIdx.x; q0 < quads; q0 += 2 * blockDim.x) {
+          const int q1 = q0 + blockDim.x;
+          const bool two = q1 < quads;
+          float4 v0 = make_float4(0, 0, 0, 0), v1 = v0;
+          const float4 w0 = gains(q0), w1 = two ? gains(q1) : v0;
+          for (int s4 = 0; s4 < p.streams; s4 += 4) {
+            float4 x0[4], x1[4];
+            float in[4];
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const int q = q0 + k * blockDim.x;
-          v[k] = wn[k] = make_float4(0, 0, 0, 0);
-          if (q < quads) {
-            if constexpr (reads_streams(EPI)) {
-              /* the weighted sum of the streams takes the place of x */
-              for (int s = 0; s < p.streams; ++s)
-                axpy(v[k], p.stream_in ? p.stream_in[s] : 1.0f,
-                     px4[s * (p.stream_stride / 4) + q]);
-            } else {
-              v[k] = px4[q];
+            for (int k = 0; k < 4; ++k) {
+              x0[k] = x1[k] = make_float4(0, 0, 0, 0);
+              in[k] = 0.0f;
+              if (s4 + k < p.streams) {
+                in[k] = p.stream_in ? p.stream_in[s4 + k] : 1.0f;
+                x0[k] = px4[(s4 + k) * next + q0];
+                if (two)
+                  x1[k] = px4[(s4 + k) * next + q1];
+              }
             }
-            if (p.norm_bf16) {
-              const uint2 w = reinterpret_cast<const uint2 *>(p.norm_w)[q];
-              wn[k] = make_float4(bf_lo(w.x), bf_hi(w.x), bf_lo(w.y), bf_hi(w.y));
-            } else {
-              wn[k] = reinterpret_cast<const float4 *>(p.norm_w)[q];
+#pragma unroll
+            for (int k = 0; k < 4; ++k) {
+              axpy(v0, in[k], x0[k]);
+              axpy(v1, in[k], x1[k]);
             }
           }
+          stage(q0, v0, w0);
+          if (two)
+            stage(q1, v1, w1);
         }
+      } else {
+        for (int q0 = threadIdx.x; q0 < quads; q0 += 4 * blockDim.x) {
+          float4 v[4], wn[4];
 #pragma unroll
-        for (int k = 0; k < 4; ++k) {
-          const int q = q0 + k * blockDim.x;
-          if (q < quads) {
-            *reinterpret_cast<float4 *>(&xs[b * xs_stride + xs_at(4 * q)]) =
-                make_float4(v[k].x * wn[k].x, v[k].y * wn[k].y, v[k].z * wn[k].z,
-                            v[k].w * wn[k].w);
-            ss = fmaf(v[k].x, v[k].x, ss);
-            ss = fmaf(v[k].y, v[k].y, ss);
-            ss = fmaf(v[k].z, v[k].z, ss);
-            ss = fmaf(v[k].w, v[k].w, ss);
+          for (int k = 0; k < 4; ++k) {
+            const int q = q0 + k * blockDim.x;
+            v[k] = wn[k] = make_float4(0, 0, 0, 0);
+            if (q < quads) {
+              v[k] = px4[q];
+              wn[k] = gains(q);
+            }
+          }
+#pragma unroll
+          for (int k = 0; k < 4; ++k) {
+            const int q = q0 + k * blockDim.x;
+            if (q < quads)
+              stage(q, v[k], wn[k]);
           }
         }
       }
