@@ -57,19 +57,29 @@ def test_ctypes_can_bind_every_symbol(built):
         assert getattr(L, name)
 
 
-def test_the_smaller_library_has_every_entry_point(built):
-    """The library that serves decoders of parallel blocks only: the same exports,
-    with refusals in place of the kernels it leaves out."""
+@pytest.mark.parametrize("kind", ["parallel", "stream"])
+def test_the_smaller_libraries_have_every_entry_point(built, kind):
+    """The libraries that serve one kind of decoder only: the same exports, with
+    refusals in place of the kernels they leave out."""
     from vx_b200 import build
-    assert build.for_parallel_decoders() == build.LIB     # the whole one is there
-    small = build._library(build.PARALLEL_LIB, build.PARALLEL_SOURCES)
+    whole, lib, sources, other, config = {
+        "parallel": (build.for_parallel_decoders, build.PARALLEL_LIB,
+                     build.PARALLEL_SOURCES, "vx_decoder_create_streams", "StreamConfig"),
+        "stream": (build.for_stream_decoders, build.STREAM_LIB, build.STREAM_SOURCES,
+                   "vx_decoder_create_parallel", "ParallelConfig"),
+    }[kind]
+    assert whole() == build.LIB     # the whole one is there
+    small = build._library(lib, sources)
     c_names = lambda path: {n for n in exported(path) if not n.startswith("_Z")}
     assert c_names(small) == c_names(built)
-    r = run_child("from vx_b200.lib import lib, use\n"
+    r = run_child("import ctypes\n"
+                  "from vx_b200.lib import lib, use, %s as Config\n"
                   "use(%r)\n"
                   "assert lib().vx_b200_gemm_q4(None, None, None, None, 1, 8, 32) == -1\n"
                   "assert b'not part of this library' in lib().vx_b200_last_error()\n"
-                  % small)
+                  "assert not lib().%s(ctypes.byref(Config()))\n"
+                  "assert b'%s is not part' in lib().vx_b200_last_error()\n"
+                  % (config, small, other, other))
     assert r.returncode == 0, r.stderr
 
 

@@ -424,20 +424,18 @@ latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
 __global__ void __launch_bounds__(256)
 latent_down_kernel(const LatentArgs a, const float *partials, int splits, int t_count,
                    int q_rank, const float *q_gain, int q_mean, __nv_bfloat16 *terms) {
-  extern __shared__ float down_row[]; /* [q_rank + kv_rank] */
+  extern __shared__ __align__(16) float down_row[]; /* [q_rank + kv_rank] */
   __shared__ float red[2][8];
   const int64_t t = blockIdx.x;
   const int tid = threadIdx.x, K = a.kv_rank, both = q_rank + K, n = both + a.rot;
   const int pos = a.positions[0] + (int)t;
   float *ring = a.ring + (int64_t)(pos % a.cache_rows) * (K + a.rot);
   float sq = 0.0f, sk = 0.0f;
-  for (int i = tid; i < both; i += 256) {
-    const float v = sum_runs(partials, splits, t_count, n, t, i);
-    down_row[i] = v;
-    if (i < q_rank)
-      sq = fmaf(v, v, sq);
-    else
-      sk = fmaf(v, v, sk);
+  for (int i = tid * 4; i < both; i += 1024) {
+    const float4 v = sum_runs4(partials, splits, t_count, n, t, i);
+    *reinterpret_cast<float4 *>(down_row + i) = v;
+    float &ss = i < q_rank ? sq : sk;
+    ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, fmaf(v.w, v.w, ss))));
   }
   sq = warp_sum(sq);
   sk = warp_sum(sk);
@@ -461,11 +459,19 @@ latent_down_kernel(const LatentArgs a, const float *partials, int splits, int t_
   }
   const float q_inv = 1.0f / sqrtf(sq / (float)q_mean + a.eps);
   const float k_inv = 1.0f / sqrtf(sk / (float)a.kv_mean + a.eps);
-  for (int i = tid; i < both; i += 256) {
-    if (i < q_rank)
-      store_terms(terms, q_rank, t, i, down_row[i] * q_inv * q_gain[i]);
+  for (int i = tid * 4; i < both; i += 1024) {
+    const float4 v = *reinterpret_cast<const float4 *>(down_row + i);
+    const bool of_q = i < q_rank;
+    const float4 g = *reinterpret_cast<const float4 *>(of_q ? q_gain + i
+                                                            : a.gain + i - q_rank);
+    const float inv = of_q ? q_inv : k_inv;
+    const float out[4] = {v.x * inv * g.x, v.y * inv * g.y, v.z * inv * g.z,
+                          v.w * inv * g.w};
+    if (of_q)
+      store_terms4(terms, q_rank, t, i, out);
     else
-      ring[i - q_rank] = down_row[i] * k_inv * a.gain[i - q_rank];
+      *reinterpret_cast<float4 *>(ring + i - q_rank) =
+          make_float4(out[0], out[1], out[2], out[3]);
   }
 }
 
