@@ -7,6 +7,7 @@ namespace vxb {
 ABSENT(rowdot_streams_f32, int, RowDotParams &, Stream)
 ABSENT(rowdot_streams_bf16, int, RowDotParams &, Stream)
 int latent_status() { return 0; }
+int gated_linear_status() { return 0; }
 int rowdot_streams_f32_status() { return 0; }
 int rowdot_streams_bf16_status() { return 0; }
 

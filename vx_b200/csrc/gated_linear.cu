@@ -200,16 +200,18 @@ gated_linear_decay_kernel(const GatedLinearArgs a, const float *in, int64_t in_s
  * LG lanes side by side hold the key channels of RJ columns (lane g of them channels
  * 4 (LG c + g) .. + 3, c below NI), so a warp holds 32 / LG * RJ columns of a head
  * and a block SCAN_WARPS times as many. q, k, alpha and v of TT positions at a time
- * come through two shared-memory buffers (past the end: q = k = v = 0, alpha = 1, which
- * leave the state as it is). Two channels go through a multiply-add together, and the
- * sums over the lanes are taken for TS positions at once. */
-constexpr int SCAN_WARPS = 8, SCAN_THREADS = SCAN_WARPS * 32, TT = 16, TS = 8;
-
-__device__ __forceinline__ void copy16(float *dst, const float *src) {
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(ptx::smem_addr(dst)),
-               "l"(src)
-               : "memory");
+ * come by bulk copies into two shared-memory buffers (past the end: q = k = v = 0,
+ * alpha = 1, which leave the state as it is), which a warp of their own asks for. Two
+ * channels go through a multiply-add together, and the sums over the lanes are taken
+ * for TS positions at once. */
+constexpr int SCAN_WARPS = 8, SCAN_THREADS = (SCAN_WARPS + 1) * 32, TS = 8;
+__host__ __device__ constexpr int scan_tile(int NI) { return NI > 2 ? 16 : 32; }
+/* floats of shared memory */
+__host__ __device__ constexpr int scan_smem(int NI, int COLS, int dim) {
+  return 2 * scan_tile(NI) * (3 * dim + COLS) + scan_tile(NI) * COLS;
 }
+
+__device__ int g_scan_status; /* 0x62: a tile never arrived; 0x63: or was never used */
 
 /* The sums of N values over the LG lanes of a group: half of the values change hands
    at every exchange while there are several, so that lane g is left with the sums of
@@ -246,45 +248,71 @@ template <int LG, int NI, int RJ>
 __global__ void __launch_bounds__(SCAN_THREADS)
 gated_linear_scan_kernel(const GatedLinearArgs a, const float *in, int64_t in_stride,
                          const float *alpha, int t_count, float *o) {
+  constexpr int TT = scan_tile(NI);
   static_assert(RJ % 4 == 0 && TT % TS == 0, "columns in fours, whole batches");
   constexpr int WARP_COLS = 32 / LG * RJ, COLS = SCAN_WARPS * WARP_COLS;
-  extern __shared__ __align__(16) float scan_smem[];
+  extern __shared__ __align__(128) float scan_shared[];
+  __shared__ __align__(8) uint64_t full[2], empty[2];
   const int dim = a.dim, vdim = a.vdim;
   const int step = 3 * dim + COLS; /* floats of a position: q | k | alpha | v */
-  float *buf = scan_smem;          /* [2][TT][step] */
-  float *so = buf + 2 * TT * step; /* [TT][COLS] */
+  float *buf = scan_shared;        /* [2][TT][step] */
+  float *so = buf + 2 * TT * step; /* [warp][TT][WARP_COLS] */
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int h = blockIdx.y, col0 = blockIdx.x * COLS;
+  const int v_cols = min(COLS, vdim - col0);
   const int g = lane % LG, group = lane / LG;
   const int mine = warp * WARP_COLS + group * RJ; /* first column, in the block */
   const Parts at(a);
   const bool fresh = a.positions[0] == 0;
   float *state = a.state + (int64_t)h * dim * vdim;
 
-  auto fetch = [&](int t0, float *to) {
-    const int quads = step / 4, dq = dim / 4, n = min(TT, t_count - t0);
-    const int filled = (n + TS - 1) / TS * TS;
-    for (int i = tid; i < filled * quads; i += SCAN_THREADS) {
-      const int t = i / quads, q = i - t * quads;
-      const float *row = in + (int64_t)(t0 + t) * in_stride;
-      float *dst = to + t * step + q * 4;
-      if (t >= n) {
-        const float v = q >= 2 * dq && q < 3 * dq ? 1.0f : 0.0f;
-        *reinterpret_cast<float4 *>(dst) = make_float4(v, v, v, v);
-      } else if (q < dq)
-        copy16(dst, row + h * dim + q * 4);
-      else if (q < 2 * dq)
-        copy16(dst, row + at.k + h * dim + (q - dq) * 4);
-      else if (q < 3 * dq)
-        copy16(dst, alpha + (int64_t)(t0 + t) * a.heads * dim + h * dim +
-                        (q - 2 * dq) * 4);
-      else if (col0 + (q - 3 * dq) * 4 < vdim)
-        copy16(dst, row + at.v + h * vdim + col0 + (q - 3 * dq) * 4);
-      else
-        *reinterpret_cast<float4 *>(dst) = make_float4(0, 0, 0, 0);
+  if (tid == 0) {
+    for (int side = 0; side < 2; ++side) {
+      ptx::mbar_init(&full[side], 1);
+      ptx::mbar_init(&empty[side], SCAN_WARPS);
     }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
+    ptx::fence_proxy_async_smem();
+    ptx::fence_barrier_init();
+  }
+  if (v_cols < COLS) /* the columns of nobody */
+    for (int i = tid; i < 2 * TT * (COLS - v_cols); i += SCAN_THREADS) {
+      const int t = i / (COLS - v_cols);
+      buf[t * step + 3 * dim + v_cols + i - t * (COLS - v_cols)] = 0.0f;
+    }
+  __syncthreads();
+
+  if (warp == SCAN_WARPS) {
+    for (int t0 = 0, tile = 0; t0 < t_count; t0 += TT, ++tile) {
+      const int side = tile & 1, n = min(TT, t_count - t0);
+      const uint32_t phase = ((tile >> 1) & 1) ^ 1;
+      if (!__all_sync(0xffffffffu, ptx::mbar_try_wait(&empty[side], phase) ||
+                                       ptx::mbar_wait_alone(&empty[side], phase))) {
+        atomicCAS(&g_scan_status, 0, 0x63);
+        break;
+      }
+      float *to = buf + side * TT * step;
+      const int filled = (n + TS - 1) / TS * TS;
+      for (int i = n * step + lane; i < filled * step; i += 32) {
+        const int c = i % step;
+        to[i] = c >= 2 * dim && c < 3 * dim ? 1.0f : 0.0f;
+      }
+      __syncwarp();
+      if (lane == 0)
+        ptx::mbar_expect_tx(&full[side], n * (3 * dim + v_cols) * (int)sizeof(float));
+      __syncwarp();
+      for (int i = lane; i < n * 4; i += 32) {
+        const int t = i >> 2, part = i & 3;
+        const float *row = in + (int64_t)(t0 + t) * in_stride;
+        const float *src = part == 0   ? row + h * dim
+                           : part == 1 ? row + at.k + h * dim
+                           : part == 2 ? alpha + ((int64_t)(t0 + t) * a.heads + h) * dim
+                                       : row + at.v + h * vdim + col0;
+        ptx::bulk_load(to + t * step + part * dim, src,
+                       (part == 3 ? v_cols : dim) * (int)sizeof(float), &full[side]);
+      }
+    }
+    return; /* the others use every tile up before they leave */
+  }
 
   float2 s[2 * NI][RJ]; /* two neighbouring channels of a column */
   auto each_cell = [&](auto body) {
@@ -299,17 +327,15 @@ gated_linear_scan_kernel(const GatedLinearArgs a, const float *in, int64_t in_st
     if (!fresh && i < dim && col < vdim)
       cell = make_float2(state[(int64_t)i * vdim + col], state[(int64_t)(i + 1) * vdim + col]);
   });
-  fetch(0, buf);
-  int side = 0;
-  for (int t0 = 0; t0 < t_count; t0 += TT, side ^= 1) {
-    const int n = min(TT, t_count - t0);
-    if (t0 + TT < t_count) {
-      fetch(t0 + TT, buf + (side ^ 1) * TT * step);
-      asm volatile("cp.async.wait_group 1;" ::: "memory");
-    } else {
-      asm volatile("cp.async.wait_group 0;" ::: "memory");
+  float *out = so + warp * TT * WARP_COLS;
+  for (int t0 = 0, tile = 0; t0 < t_count; t0 += TT, ++tile) {
+    const int side = tile & 1, n = min(TT, t_count - t0);
+    const uint32_t phase = (tile >> 1) & 1;
+    if (!__all_sync(0xffffffffu, ptx::mbar_try_wait(&full[side], phase) ||
+                                     ptx::mbar_wait_alone(&full[side], phase))) {
+      atomicCAS(&g_scan_status, 0, 0x62);
+      break;
     }
-    __syncthreads();
     const float *now = buf + side * TT * step;
     for (int t = 0; t < n; t += TS) {
       float part[TS * RJ];
@@ -359,16 +385,21 @@ gated_linear_scan_kernel(const GatedLinearArgs a, const float *in, int64_t in_st
       if (owner)
 #pragma unroll
         for (int j = 0; j < LEFT; ++j)
-          so[(t + (one + j) / RJ) * COLS + mine + (one + j) % RJ] = part[j] * a.q_scale;
+          out[(t + (one + j) / RJ) * WARP_COLS + group * RJ + (one + j) % RJ] =
+              part[j] * a.q_scale;
     }
-    __syncthreads(); /* the buffer may be filled again; so is complete */
-    for (int i = tid; i < n * (COLS / 4); i += SCAN_THREADS) {
-      const int t = i / (COLS / 4), c = i % (COLS / 4) * 4;
-      if (col0 + c < vdim)
+    __syncwarp();
+    if (lane == 0)
+      ptx::mbar_arrive(&empty[side]);
+    for (int i = lane; i < n * (WARP_COLS / 4); i += 32) {
+      const int t = i / (WARP_COLS / 4), c = i % (WARP_COLS / 4) * 4;
+      const int col = col0 + warp * WARP_COLS + c;
+      if (col < vdim)
         *reinterpret_cast<float4 *>(o + (int64_t)(t0 + t) * a.heads * vdim + h * vdim +
-                                    col0 + c) =
-            *reinterpret_cast<const float4 *>(&so[t * COLS + c]);
+                                    col) =
+            *reinterpret_cast<const float4 *>(&out[t * WARP_COLS + c]);
     }
+    __syncwarp();
   }
   each_cell([&](float2 &cell, int i, int col) {
     if (i < dim && col < vdim) {
@@ -420,9 +451,8 @@ template <int LG, int NI, int RJ>
 const char *launch_scan(const GatedLinearArgs &a, const float *in, int64_t in_stride,
                         const float *alpha, int t, float *o, cudaStream_t stream) {
   constexpr int COLS = SCAN_WARPS * 32 / LG * RJ;
-  const int smem = (2 * TT * (3 * a.dim + COLS) + TT * COLS) * (int)sizeof(float);
-  constexpr int most =
-      (2 * TT * (3 * LG * NI * 4 + COLS) + TT * COLS) * (int)sizeof(float);
+  const int smem = scan_smem(NI, COLS, a.dim) * (int)sizeof(float);
+  constexpr int most = scan_smem(NI, COLS, LG * NI * 4) * (int)sizeof(float);
   static_assert(most <= 227 * 1024, "the buffers fit in shared memory");
   const void *kernel = (const void *)gated_linear_scan_kernel<LG, NI, RJ>;
   if (allow_dynamic_smem(kernel, most) != cudaSuccess)
@@ -477,6 +507,15 @@ const char *gated_linear_scan(const GatedLinearArgs &a, const float *in, int64_t
   if (a.dim <= 256)
     return launch_scan<32, 2, 4>(a, in, in_stride, alpha, t, o, stream);
   return launch_scan<32, 4, 4>(a, in, in_stride, alpha, t, o, stream);
+}
+
+int gated_linear_status() {
+  int v = 0, zero = 0;
+  if (cudaMemcpyFromSymbol(&v, g_scan_status, sizeof v) != cudaSuccess)
+    return -1;
+  if (v)
+    cudaMemcpyToSymbol(g_scan_status, &zero, sizeof zero);
+  return v;
 }
 
 const char *gated_linear_finish(const GatedLinearArgs &a, const float *in,

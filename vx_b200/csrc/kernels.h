@@ -617,6 +617,7 @@ const char *gated_linear_decays(const GatedLinearArgs &a, const float *in,
                                 cudaStream_t stream);
 const char *gated_linear_scan(const GatedLinearArgs &a, const float *in, int64_t in_stride,
                               const float *alpha, int t, float *o, cudaStream_t stream);
+int gated_linear_status(); /* 0, or once the code of a copy that did not arrive */
 /* Norm and gate of o, as terms in the first columns of [t][3 cols]. */
 const char *gated_linear_finish(const GatedLinearArgs &a, const float *in,
                                 int64_t in_stride, const float *o, int t, void *terms,

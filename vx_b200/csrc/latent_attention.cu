@@ -262,8 +262,8 @@ latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
       if (j < have) {
         uint64_t *bar = &bars[warp][slot];
         const uint32_t phase = (j / SLOTS) & 1;
-        arrived = arrived &&
-                  (ptx::mbar_try_wait(bar, phase) || ptx::mbar_wait_alone(bar, phase));
+        arrived = arrived && __all_sync(0xffffffffu, ptx::mbar_try_wait(bar, phase) ||
+                                                         ptx::mbar_wait_alone(bar, phase));
         src = my_slots + slot * ROW;
       }
 #pragma unroll

@@ -1097,7 +1097,8 @@ int32_t vx_b200_kernel_status(void) {
   const int s = vxb::step_status(vxb::caller_stream());
   const int e = vxb::moe_group_status(vxb::caller_stream());
   const int l = vxb::latent_status();
-  return g ? g : (f ? f : (t ? t : (m ? m : (r ? r : (s ? s : (e ? e : l))))));
+  const int c = vxb::gated_linear_status();
+  return g ? g : (f ? f : (t ? t : (m ? m : (r ? r : (s ? s : (e ? e : (l ? l : c)))))));
 }
 
 int32_t vx_b200_attention_kernel(int32_t which) {
