@@ -421,7 +421,7 @@ latent_decode_kernel(const LatentArgs a, const float *q_in, int64_t q_stride,
 
 /* ---- the positions of a prompt: the ring's rows and the query latent -------------
  * A block is a position. */
-__global__ void __launch_bounds__(256)
+__global__ void __launch_bounds__(256, 6)
 latent_down_kernel(const LatentArgs a, const float *partials, int splits, int t_count,
                    int q_rank, const float *q_gain, int q_mean, __nv_bfloat16 *terms) {
   extern __shared__ __align__(16) float down_row[]; /* [q_rank + kv_rank] */
@@ -442,14 +442,6 @@ latent_down_kernel(const LatentArgs a, const float *partials, int splits, int t_
   if ((tid & 31) == 0) {
     red[0][tid >> 5] = sq;
     red[1][tid >> 5] = sk;
-  }
-  for (int k = tid; k < a.rot / 2; k += 256) {
-    const float u = sum_runs(partials, splits, t_count, n, t, both + 2 * k);
-    const float v = sum_runs(partials, splits, t_count, n, t, both + 2 * k + 1);
-    float sine, cosine;
-    turned(pos, a.turns[k], sine, cosine);
-    ring[K + 2 * k] = u * cosine - v * sine;
-    ring[K + 2 * k + 1] = v * cosine + u * sine;
   }
   __syncthreads();
   sq = sk = 0.0f;
@@ -472,6 +464,15 @@ latent_down_kernel(const LatentArgs a, const float *partials, int splits, int t_
     else
       *reinterpret_cast<float4 *>(ring + i - q_rank) =
           make_float4(out[0], out[1], out[2], out[3]);
+  }
+  /* the rotated part, by the warps that have least of the rest */
+  for (int k = 255 - tid; k < a.rot / 2; k += 256) {
+    const float u = sum_runs(partials, splits, t_count, n, t, both + 2 * k);
+    const float v = sum_runs(partials, splits, t_count, n, t, both + 2 * k + 1);
+    float sine, cosine;
+    turned(pos, a.turns[k], sine, cosine);
+    ring[K + 2 * k] = u * cosine - v * sine;
+    ring[K + 2 * k + 1] = v * cosine + u * sine;
   }
 }
 
